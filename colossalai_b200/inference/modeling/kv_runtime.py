@@ -124,11 +124,11 @@ class PagedKVRuntime:
                       bias_table=None, bucket_starts=None, sink: bool = False, v_other=None,
                       lam: float = 0.0, lut=None, mask_block: int = 0, wide_weights: bool = False,
                       sink_values: Optional[torch.Tensor] = None, slopes: Optional[torch.Tensor] = None,
-                      window: int = 0) -> torch.Tensor:
+                      window: int = 0, keep_first: int = 0) -> torch.Tensor:
         """Write the step's K / V rows (values optionally blended with `v_other`) into the layer's pages, then attend
         every step token over positions 0..pos of its sequence (with `mask_block`: over the positions of its own block
-        of that many positions only; with `window`: over the last `window` positions; `slopes`: a linear distance
-        penalty per head; `sink_values`: the sink's score per head).  q [T, H x dim], k [T, G x dim], v [T, G x vdim];
+        of that many positions only; with `window`: over the last `window` positions, with `keep_first` also over the
+        first that many of the sequence; `slopes`: a linear distance penalty per head; `sink_values`: the sink's score per head).  q [T, H x dim], k [T, G x dim], v [T, G x vdim];
         k = None: the caller has written the step's rows itself (`pages`)."""
         from ...ops import mixers as mops
 
@@ -137,7 +137,8 @@ class PagedKVRuntime:
             mops.paged_kv_write_mix(k, v, kc, vc, self.block_tables, self.ragged, v_other=v_other, lam=lam)
         return mops.paged_bias_attention(q, kc, vc, self.block_tables, self.ragged, scale, bias_table=bias_table,
                                          bucket_starts=bucket_starts, sink=sink, lut=lut, mask_block=mask_block,
-                                         wide_weights=wide_weights, sink_values=sink_values, slopes=slopes, window=window)
+                                         wide_weights=wide_weights, sink_values=sink_values, slopes=slopes, window=window,
+                                         keep_first=keep_first)
 
     @classmethod
     def scratch(cls, cfg, batch: int, seqlen: int, device, dtype, block_size: int = 16) -> "PagedKVRuntime":

@@ -37,6 +37,9 @@
 //   cb_paged_bias_attention causal attention of every step token over its sequence's paged cache with
 //                           score = scale * q.k + table[bucket(distance)][head] - slope[head] * distance, an optional
 //                           sink (score 0 or learned per head) in the denominator, a block mask or a sliding window
+//   cb_stream_tanh_norm     x(fp32) += y or n_o(y);  h = cast(n_i(x)), n(z) = tanh(alpha z) w + b element by element
+//   cb_router_sigmoid       sigmoid router scores, choice by score + correction inside the best groups of experts
+//   cb_rotary_kv_write      q heads rotated in place, rotated k heads and v heads into their pages, one pass over q | k | v
 //   cb_depth_mix            weighted sum over the history of the fp32 stream (+ compute-dtype copy)
 //   cb_poly_norm            a N(z) + b N(z^2) + c N(z^3) + e with N = division by the row's root mean square
 //   cb_head_rmsnorm         RMS norm per head with a weight over the head's channels (query heads | key heads); optionally
@@ -1274,8 +1277,16 @@ __global__ void __launch_bounds__(128) paged_kv_write_mix_kernel(const T* __rest
 // (lane = key for the scores, lane = value channel for the weighted sum), online softmax in fp32.  With `sink` the running
 // maximum starts at the sink's score (`sink_vals[head]`, 0 without the table) and the denominator at 1: a key of that
 // score without a value, not scaled.  `slopes[head]` takes slope * (pos - key) off every score; `window` > 0 keeps the
-// keys pos - window + 1 .. pos only.
+// keys pos - window + 1 .. pos and, whatever their distance, the first `keep_first` keys of the sequence.
 constexpr int ATT_MAX_VREG = 16;  // value width up to 512
+
+// first key of the contiguous range that ends at position p: the start of p's own block (block mask), the first key of
+// p's window, or 0
+CB_DEVICE int att_first_key(int p, int mask_block, int window) {
+  int f = mask_block > 0 ? p / mask_block * mask_block : 0;
+  if (window > 0) f = max(f, p - window + 1);
+  return f;
+}
 
 template <typename T>
 __global__ void __launch_bounds__(128) paged_bias_attention_kernel(
@@ -1283,7 +1294,8 @@ __global__ void __launch_bounds__(128) paged_bias_attention_kernel(
     const int* __restrict__ block_tables, const int* __restrict__ token_seq, const int* __restrict__ token_pos,
     const float* __restrict__ bias_table, const int* __restrict__ bucket_start, int nbuckets, T* __restrict__ out,
     int64_t tokens, int heads, int kv_heads, int dim, int vdim, int ldv, int block_size, int max_blocks, float scale,
-    int sink, int mask_block, const float* __restrict__ sink_vals, const float* __restrict__ slopes, int window) {
+    int sink, int mask_block, const float* __restrict__ sink_vals, const float* __restrict__ slopes, int window,
+    int keep_first) {
   extern __shared__ float smem[];
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
   float* qs = smem + warp * dim;
@@ -1305,14 +1317,16 @@ __global__ void __launch_bounds__(128) paged_bias_attention_kernel(
   float acc[ATT_MAX_VREG];
 #pragma unroll
   for (int r = 0; r < ATT_MAX_VREG; ++r) acc[r] = 0.f;
-  // with a block mask the keys start at the first position of the query's own block, with a window at its first key
-  int jfirst = mask_block > 0 ? pos / mask_block * mask_block : 0;
-  if (window > 0) jfirst = max(jfirst, pos - window + 1);
-  for (int j0 = jfirst; j0 <= pos; j0 += 32) {
-    const int jk = j0 + lane;
+  // the visible keys, numbered without gaps: the kept first ones that lie in front of the range, then jfirst .. pos
+  const int jfirst = att_first_key(pos, mask_block, window);
+  const int kept = min(keep_first, jfirst);
+  const int nkeys = kept + pos - jfirst + 1;
+  for (int n0 = 0; n0 < nkeys; n0 += 32) {
+    const int nth = n0 + lane;
+    const int jk = nth < kept ? nth : jfirst + nth - kept;
     float sc = -INFINITY;
     int64_t myrow = 0;
-    if (jk <= pos) {
+    if (nth < nkeys) {
       myrow = ((int64_t)bt[jk / block_size] * block_size + jk % block_size) * kv_heads + g;
       const T* kr = k_cache + myrow * dim;
       float d0 = 0.f, d1 = 0.f;
@@ -1336,12 +1350,12 @@ __global__ void __launch_bounds__(128) paged_bias_attention_kernel(
     }
     const float mn = fmaxf(m, warp_max(sc));
     const float alpha = expf(m - mn);           // m = -inf only before the first tile without a sink: exp(-inf) = 0
-    const float pj = jk <= pos ? expf(sc - mn) : 0.f;
+    const float pj = nth < nkeys ? expf(sc - mn) : 0.f;
     l = l * alpha + warp_sum(pj);
     m = mn;
 #pragma unroll
     for (int r = 0; r < ATT_MAX_VREG; ++r) acc[r] *= alpha;
-    const int nk = min(32, pos - j0 + 1);
+    const int nk = min(32, nkeys - n0);
     for (int jj = 0; jj < nk; ++jj) {
       const float pw = __shfl_sync(0xffffffffu, pj, jj);
       const int64_t vrow = __shfl_sync(0xffffffffu, myrow, jj);
@@ -1408,14 +1422,21 @@ CB_DEVICE void cp_async16(void* smem_dst, const void* gmem_src, uint32_t src_byt
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(gmem_src), "r"(src_bytes) : "memory");
 }
 
-// Key range split (decode steps, few CTAs): with `chunk` > 0 grid.x also enumerates key chunks; a CTA then writes its
-// unnormalised partial (fp32 accumulator, running maximum, denominator without the sink) and `attention_merge_kernel`
-// joins the chunks of every (token, head) in ascending order.
+// A row tile walks a list of 64-key tiles: those that hold kept first keys in front of its rows' ranges (`keep_first`,
+// `att_kept_tiles` of them), then the tiles from its first row's first key to its last row's position.  With a window the
+// list is short whatever the context's length.
+//
+// Key range split (decode steps, few CTAs): with `chunk` > 0 grid.x also enumerates chunks of chunk / 64 tiles of that
+// list; a CTA then writes its unnormalised partial (fp32 accumulator, running maximum, denominator without the sink) and
+// `attention_merge_kernel` joins the chunks of every (token, head) in ascending order.
 //
 // A CTA is 4 warps x 32 rows (MT = 2 m16 tiles per warp) when a portion fills 128 rows, 4 x 16 (MT = 1) otherwise.  Two
 // m-tiles per warp halve the shared-memory reads per MMA (a K / V fragment feeds both) and double the independent
 // accumulator chains.  The query tile sits in shared memory (A fragments by ldmatrix.x4, K fragments by ldmatrix.x4
 // for two k-steps at once, V fragments by ldmatrix.x2.trans).
+CB_DEVICE int att_kept_tiles(int keep_first, int blk_lo) {
+  return min((keep_first + MMA_BN - 1) / MMA_BN, blk_lo / MMA_BN);
+}
 CB_DEVICE void ldsm_x4(uint32_t (&r)[4], uint32_t addr) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
                : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
@@ -1432,7 +1453,7 @@ __global__ void __launch_bounds__(128, D > 128 ? 1 : (MT == 2 ? 2 : 3)) paged_bi
     const float* __restrict__ bias_table, const uint8_t* __restrict__ lut, int lut_n, int nbuckets, T* __restrict__ out,
     int heads, int kv_heads, int dim, int vdim, int ldv, int block_size, int max_blocks, float scale, int sink, int chunk,
     int max_splits, float* __restrict__ part_o, float* __restrict__ part_ml, int mask_block, int wide_weights,
-    const float* __restrict__ sink_vals, const float* __restrict__ slopes, int window) {
+    const float* __restrict__ sink_vals, const float* __restrict__ slopes, int window, int keep_first) {
   constexpr int BM = 64 * MT;
   constexpr int LDS = D + 8;                    // padded row: 16-byte aligned, conflict-free fragment reads
   constexpr int TILE = MMA_BN * LDS;
@@ -1456,20 +1477,20 @@ __global__ void __launch_bounds__(128, D > 128 ? 1 : (MT == 2 ? 2 : 3)) paged_bi
   if (row0 >= nrows) return;
   const int ctx = ctx_len[s];
   const int last_row = min(nrows - 1, row0 + BM - 1);
-  // block mask: a row at position p sees keys p / mask_block * mask_block .. p; the tile's keys start at its first row's
-  // block (key chunks that end below it are never read: the merge starts at the row's own first chunk)
-  // (rounded down to a key tile, so that tiles keep their place inside a key chunk and never reach into the next one)
-  // A window of `window` positions moves a row's first key to pos - window + 1 in the same way (both grow with pos).
-  auto first_key = [&](int p) {
-    int f = mask_block > 0 ? p / mask_block * mask_block : 0;
-    if (window > 0) f = max(f, p - window + 1);
-    return f;
-  };
+  // block mask: a row at position p sees keys p / mask_block * mask_block .. p; a window of `window` positions moves a
+  // row's first key to pos - window + 1.  Both grow with pos: the tile's range starts at its first row's first key,
+  // rounded down to a key tile
   const bool masked_lo = mask_block > 0 || window > 0;
-  const int blk_lo = masked_lo ? first_key(ctx + row0 / R) / MMA_BN * MMA_BN : 0;
-  const int key_lo = max(chunk > 0 ? split * chunk : 0, blk_lo);
-  const int pos_max = chunk > 0 ? min(ctx + last_row / R, split * chunk + chunk - 1) : ctx + last_row / R;
-  if (key_lo > pos_max) return;                 // this chunk lies beyond (or below) every row of the tile
+  const int blk_lo = masked_lo ? att_first_key(ctx + row0 / R, mask_block, window) / MMA_BN * MMA_BN : 0;
+  const int pos_max = ctx + last_row / R;
+  const int nkept = att_kept_tiles(keep_first, blk_lo);
+  int vt = 0, vt_end = nkept + (pos_max - blk_lo) / MMA_BN + 1;           // the tile list; a split CTA takes a part of it
+  if (chunk > 0) {
+    vt = split * (chunk / MMA_BN);
+    vt_end = min(vt_end, vt + chunk / MMA_BN);
+  }
+  if (vt >= vt_end) return;                     // this chunk lies beyond every row of the tile
+  auto tile_key = [&](int v) { return v < nkept ? v * MMA_BN : blk_lo + (v - nkept) * MMA_BN; };
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, gid = lane >> 2, tig = lane & 3;
   for (int i = tid; i < nbuckets * R; i += 128) tab[i] = bias_table[(i / R) * heads + g * R + (i % R)] * LOG2E;
   const int* bt = block_tables + (int64_t)s * max_blocks;
@@ -1499,7 +1520,7 @@ __global__ void __launch_bounds__(128, D > 128 ? 1 : (MT == 2 ? 2 : 3)) paged_bi
                  in ? 16u : 0u);
     }
   }
-  load_tile(0, key_lo);
+  load_tile(0, tile_key(vt));
 
   int rr[NR], pos[NR], hr[NR], lo[NR];
   bool valid[NR];
@@ -1509,7 +1530,7 @@ __global__ void __launch_bounds__(128, D > 128 ? 1 : (MT == 2 ? 2 : 3)) paged_bi
     valid[e] = rr[e] < nrows;
     hr[e] = valid[e] ? rr[e] % R : 0;
     pos[e] = valid[e] ? ctx + rr[e] / R : -1;
-    lo[e] = (masked_lo && valid[e]) ? first_key(pos[e]) : 0;      // first key the row sees
+    lo[e] = (masked_lo && valid[e]) ? att_first_key(pos[e], mask_block, window) : 0;      // first key of the row's range
   }
   float o[MT][D / 8][4];
 #pragma unroll
@@ -1534,14 +1555,15 @@ __global__ void __launch_bounds__(128, D > 128 ? 1 : (MT == 2 ? 2 : 3)) paged_bi
   const bool wlive = wrow0 < nrows;
   const int wlo = ctx + min(nrows - 1, wrow0) / R;
   const int whi = wlive ? ctx + min(nrows - 1, wrow0 + 16 * MT - 1) / R : -1;
-  const int wblk = (masked_lo && wlive) ? first_key(whi) : 0;     // latest first key among its rows
+  const int wblk = (masked_lo && wlive) ? att_first_key(whi, mask_block, window) : 0;     // latest first key among its rows
   const uint32_t q_addr = (uint32_t)__cvta_generic_to_shared(Qs + ((KS ? 0 : warp * 16 * MT) + (lane & 15)) * LDS +
                                                              (lane >> 4) * 8);
 
   int stage = 0;
-  for (int j0 = key_lo; j0 <= pos_max; j0 += MMA_BN, stage ^= 1) {
-    if (j0 + MMA_BN <= pos_max) {               // the other stage was released by the barrier that ended the last pass
-      load_tile(stage ^ 1, j0 + MMA_BN);
+  for (; vt < vt_end; ++vt, stage ^= 1) {
+    const int j0 = tile_key(vt);
+    if (vt + 1 < vt_end) {                      // the other stage was released by the barrier that ended the last pass
+      load_tile(stage ^ 1, tile_key(vt + 1));
       asm volatile("cp.async.wait_group 1;" ::: "memory");
     } else {
       asm volatile("cp.async.wait_group 0;" ::: "memory");
@@ -1578,7 +1600,7 @@ __global__ void __launch_bounds__(128, D > 128 ? 1 : (MT == 2 ? 2 : 3)) paged_bi
         }
       }
       const int jlast = j0 + koff + NT * 8 - 1;  // last key this warp scores in the tile
-      const bool unmasked = jlast <= wlo && j0 + koff >= wblk;
+      const bool unmasked = jlast <= wlo && (j0 + koff >= wblk || jlast < keep_first);
       const bool far = nbuckets == 0 || wlo - jlast >= lut_n;                 // every distance in the last bucket
       float fb[NR];
 #pragma unroll
@@ -1608,7 +1630,7 @@ __global__ void __launch_bounds__(128, D > 128 ? 1 : (MT == 2 ? 2 : 3)) paged_bi
             for (int e = 0; e < 4; ++e) {
               const int r = mt * 2 + (e >> 1), j = j0 + koff + nt * 8 + tig * 2 + (e & 1);
               float sv = -INFINITY;
-              if (j <= pos[r] && j >= lo[r]) {
+              if (j <= pos[r] && (j >= lo[r] || j < keep_first)) {
                 sv = sacc[mt][nt][e] * sc2;
                 if (nbuckets > 0) {
                   const int n = pos[r] - j;
@@ -1766,27 +1788,34 @@ __global__ void __launch_bounds__(128, D > 128 ? 1 : (MT == 2 ? 2 : 3)) paged_bi
   }
 }
 
-// one warp per (token, head, 32 value columns): joins the key chunks 0..pos / chunk (log2-domain maxima).  The chunks'
+// one warp per (token, head, 32 value columns): joins the key chunks of the row's tile list (log2-domain maxima).  The
+// list belongs to the row TILE (bm rows) that the row sat in, so its start is recomputed from the tile's first row.  The chunks'
 // maxima and denominators are read with one chunk per lane and reduced over the warp; the weighted sum of the partial
 // outputs then walks the chunks in ascending order with the weights passed by shuffle, eight chunks' loads in flight.
 template <typename T>
 __global__ void __launch_bounds__(128) attention_merge_kernel(const float* __restrict__ part_o,
                                                               const float* __restrict__ part_ml,
-                                                              const int* __restrict__ token_pos, T* __restrict__ out,
-                                                              int64_t tokens, int heads, int vdim, int chunk,
-                                                              int max_splits, int sink, int mask_block,
-                                                              const float* __restrict__ sink_vals, int window) {
+                                                              const int* __restrict__ token_pos,
+                                                              const int* __restrict__ token_seq,
+                                                              const int* __restrict__ cu_q, T* __restrict__ out,
+                                                              int64_t tokens, int heads, int kv_heads, int vdim, int bm,
+                                                              int chunk, int max_splits, int sink, int mask_block,
+                                                              const float* __restrict__ sink_vals, int window,
+                                                              int keep_first) {
   const int lane = threadIdx.x & 31;
   const int cblocks = (vdim + 31) >> 5;
   const int64_t item = (int64_t)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   if (item >= tokens * heads * cblocks) return;
   const int64_t unit = item / cblocks;
   const int c = (int)(item % cblocks) * 32 + lane;
-  const int tpos = token_pos[unit / heads];
-  const int nsp = tpos / chunk + 1;
-  int kfirst = mask_block > 0 ? tpos / mask_block * mask_block : 0;
-  if (window > 0) kfirst = max(kfirst, tpos - window + 1);
-  const int sp0 = kfirst / chunk;                                                     // first chunk with a visible key
+  const int tok = (int)(unit / heads), R = heads / kv_heads, ct = chunk / MMA_BN;
+  const int tpos = token_pos[tok], nth = tok - cu_q[token_seq[tok]];                  // place in its sequence's portion
+  const int row0 = (nth * R + (int)(unit % heads) % R) / bm * bm;
+  const int blk_lo = att_first_key(tpos - nth + row0 / R, mask_block, window) / MMA_BN * MMA_BN;
+  const int nkept = att_kept_tiles(keep_first, blk_lo);
+  const int nsp = min((nkept + (tpos - blk_lo) / MMA_BN) / ct + 1, max_splits);
+  // first chunk with a visible key
+  const int sp0 = nkept > 0 ? 0 : (att_first_key(tpos, mask_block, window) - blk_lo) / MMA_BN / ct;
   const float* ml = part_ml + unit * max_splits * 2;
   const float sk = sink_vals != nullptr ? sink_vals[unit % heads] * 1.4426950408889634f : 0.f;
   float mm = sink ? sk : -INFINITY;
@@ -1813,11 +1842,12 @@ __global__ void __launch_bounds__(128) attention_merge_kernel(const float* __res
 
 template <typename T, int D, int MT, bool KS = false>
 int launch_attention_mma(const void* q, int64_t ldq, const void* k_cache, const void* v_cache, const int* block_tables,
-                         const int* cu_q, const int* ctx_len, const int* token_pos, const float* bias_table,
-                         const uint8_t* lut, int lut_n, int nbuckets, void* out, int64_t tokens, int nseq, int max_q,
+                         const int* cu_q, const int* ctx_len, const int* token_pos, const int* token_seq,
+                         const float* bias_table, const uint8_t* lut, int lut_n, int nbuckets, void* out, int64_t tokens, int nseq, int max_q,
                          int heads, int kv_heads, int dim, int vdim, int ldv, int block_size, int max_blocks, float scale,
                          int sink, int chunk, int max_splits, float* part_o, float* part_ml, int mask_block,
-                         int wide_weights, const float* sink_vals, const float* slopes, int window, cudaStream_t st) {
+                         int wide_weights, const float* sink_vals, const float* slopes, int window, int keep_first,
+                         cudaStream_t st) {
   const int R = heads / kv_heads;
   constexpr int BM = 64 * MT;
   const bool kv_same = v_cache == k_cache && ldv == dim;
@@ -1835,12 +1865,13 @@ int launch_attention_mma(const void* q, int64_t ldq, const void* k_cache, const 
   kern<<<grid, 128, smem, st>>>((const T*)q, ldq, (const T*)k_cache, (const T*)v_cache, block_tables, cu_q, ctx_len,
                                 bias_table, lut, lut_n, nbuckets, (T*)out, heads, kv_heads, dim, vdim, ldv, block_size,
                                 max_blocks, scale, sink, chunk, max_splits, part_o, part_ml, mask_block, wide_weights,
-                                sink_vals, slopes, window);
+                                sink_vals, slopes, window, keep_first);
   if (chunk > 0) {
     const int64_t units = tokens * heads * ((vdim + 31) / 32);
-    attention_merge_kernel<T><<<(unsigned)((units + 3) / 4), 128, 0, st>>>(part_o, part_ml, token_pos, (T*)out, tokens,
-                                                                          heads, vdim, chunk, max_splits, sink, mask_block,
-                                                                          sink_vals, window);
+    attention_merge_kernel<T><<<(unsigned)((units + 3) / 4), 128, 0, st>>>(part_o, part_ml, token_pos, token_seq, cu_q,
+                                                                          (T*)out, tokens, heads, kv_heads, vdim, BM, chunk,
+                                                                          max_splits, sink, mask_block, sink_vals, window,
+                                                                          keep_first);
   }
   return CB_LAUNCH_CHECK();
 }
@@ -2104,6 +2135,186 @@ __global__ void __launch_bounds__(256) sigmoid_gate_mul_kernel(T* __restrict__ o
 #pragma unroll
     for (int e = 0; e < VEC; ++e) ov[e] *= sigmoid_f(gv[e]);
     store_vec<T, VEC>(o, false, t * C + c, ov);
+  }
+}
+
+// ------------------------------------------------------------------------------------------------ tanh norms of the stream
+// n(z) = tanh(alpha z) w + b with a scalar alpha and vectors w, b (fp32 or T): no statistics over the row, so the norm of a
+// sublayer's output, its addition to the fp32 stream and the norm in front of the next sublayer are one elementwise pass.
+// A thread keeps the parameters of its VEC columns in registers and walks over the rows, TANH_ROWS of them in flight.
+constexpr int TANH_ROWS = 2;
+
+struct TanhNorm {
+  const void *alpha, *w, *b;    // w == nullptr: absent
+  int f32;
+};
+
+template <typename T, int VEC> struct TanhParams {
+  float a, w[VEC], b[VEC];
+  bool on;
+  CB_DEVICE void load(const TanhNorm& n, int c) {
+    on = n.w != nullptr;
+    if (!on) return;
+    a = n.f32 ? *(const float*)n.alpha : to_f32<T>(*(const T*)n.alpha);
+    load_vec<T, VEC>(n.w, n.f32 != 0, c, w);
+    load_vec<T, VEC>(n.b, n.f32 != 0, c, b);
+  }
+  CB_DEVICE float operator()(float z, int e) const { return fmaf(tanhf(a * z), w[e], b[e]); }
+};
+
+template <typename T, int VEC>
+__global__ void __launch_bounds__(128) stream_tanh_norm_kernel(float* __restrict__ x, const void* __restrict__ y,
+                                                               int64_t ldy, int y_f32, TanhNorm no, TanhNorm ni,
+                                                               void* __restrict__ h, int h_f32, int64_t tokens, int W) {
+  const int c = (blockIdx.x * blockDim.x + threadIdx.x) * VEC;
+  if (c >= W) return;
+  TanhParams<T, VEC> po, pi;
+  po.load(no, c);
+  pi.load(ni, c);
+  for (int64_t t0 = (int64_t)blockIdx.y * TANH_ROWS; t0 < tokens; t0 += (int64_t)gridDim.y * TANH_ROWS) {
+    float xv[TANH_ROWS][VEC], yv[TANH_ROWS][VEC];
+#pragma unroll
+    for (int r = 0; r < TANH_ROWS; ++r)
+      if (t0 + r < tokens) {
+        load_vec<T, VEC>(x, true, (t0 + r) * W + c, xv[r]);
+        if (y != nullptr) load_vec<T, VEC>(y, y_f32 != 0, (t0 + r) * ldy + c, yv[r]);
+      }
+#pragma unroll
+    for (int r = 0; r < TANH_ROWS; ++r)
+      if (t0 + r < tokens) {
+        if (y != nullptr) {
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) xv[r][e] += po.on ? po(yv[r][e], e) : yv[r][e];
+          store_vec<T, VEC>(x, true, (t0 + r) * W + c, xv[r]);
+        }
+        if (pi.on) {
+          float hv[VEC];
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) hv[e] = pi(xv[r][e], e);
+          store_vec<T, VEC>(h, h_f32 != 0, (t0 + r) * W + c, hv);
+        }
+      }
+  }
+}
+
+// ------------------------------------------------------------------------------------------------ router
+// One warp per token: s = sigmoid(z), choice score c = s + correction.  Experts form `groups` equal groups of neighbours; a
+// group's score is the sum of its two largest choice scores, and only the experts of the `keep` best groups (ties: the
+// lower index) can be chosen.  The K largest choice scores win, their weights are s itself (renormalised with `renorm`).
+constexpr int ROUTER_WARPS = 4;
+
+__global__ void __launch_bounds__(ROUTER_WARPS * 32) router_sigmoid_kernel(const float* __restrict__ logits, int64_t ldz,
+                                                                           const float* __restrict__ corr,
+                                                                           float* __restrict__ w_out,
+                                                                           int64_t* __restrict__ idx_out, int64_t tokens,
+                                                                           int E, int K, int groups, int keep, int renorm) {
+  extern __shared__ float router_smem[];
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  float* c = router_smem + warp * (E + groups);             // choice scores [E], then group scores [groups]
+  float* gs = c + E;
+  const int64_t t = (int64_t)blockIdx.x * ROUTER_WARPS + warp;
+  if (t >= tokens) return;
+  const float* z = logits + t * ldz;
+  for (int e = lane; e < E; e += 32) c[e] = sigmoid_f(z[e]) + (corr != nullptr ? corr[e] : 0.f);
+  __syncwarp();
+  if (keep < groups) {
+    const int n = E / groups;
+    for (int g = lane; g < groups; g += 32) {
+      float a = -INFINITY, b = -INFINITY;                   // largest, second largest
+      for (int i = 0; i < n; ++i) {
+        const float v = c[g * n + i];
+        if (v > a) { b = a; a = v; } else if (v > b) b = v;
+      }
+      gs[g] = n > 1 ? a + b : a;
+    }
+    __syncwarp();
+    for (int e = lane; e < E; e += 32) {
+      const int g = e / n;
+      int better = 0;
+      for (int o = 0; o < groups; ++o) better += gs[o] > gs[g] || (gs[o] == gs[g] && o < g);
+      if (better >= keep) c[e] = -INFINITY;
+    }
+    __syncwarp();
+  }
+  float sum = 0.f;
+  for (int k = 0; k < K; ++k) {
+    float best = -INFINITY;
+    int bi = 0x7fffffff;
+    for (int e = lane; e < E; e += 32)
+      if (c[e] > best) { best = c[e]; bi = e; }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+      const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+      if (ob > best || (ob == best && oi < bi)) { best = ob; bi = oi; }
+    }
+    bi = min(bi, E - 1);                                    // (no comparable score left: NaN logits)
+    const float s = sigmoid_f(z[bi]);
+    sum += s;
+    if (lane == 0) {
+      w_out[t * K + k] = s;
+      idx_out[t * K + k] = bi;
+      c[bi] = -INFINITY;
+    }
+    __syncwarp();
+  }
+  if (renorm)
+    for (int k = lane; k < K; k += 32) w_out[t * K + k] /= fmaxf(sum, 1e-20f);
+}
+
+// ------------------------------------------------------------------------------------------------ rotary q | k | v
+// One pass over the projection rows q | k | v: the rotated channels of the query heads are turned in place (the others stay
+// where they are), the key heads go rotated into their pages, the value heads into theirs.  A work item is VEC channels: in
+// the rotated part VEC channels of the first half together with their partners.  A CTA takes as many tokens as it has
+// threads for.
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256) rotary_kv_write_kernel(T* __restrict__ qkv, int64_t ld, int64_t tokens, int H, int G,
+                                                              int dim, int vdim, int rot, const float* __restrict__ table,
+                                                              T* __restrict__ k_cache, T* __restrict__ v_cache,
+                                                              const int* __restrict__ block_tables,
+                                                              const int* __restrict__ token_seq,
+                                                              const int* __restrict__ token_pos, int block_size,
+                                                              int max_blocks, int tok_per_cta) {
+  struct alignas(sizeof(T) * VEC) Pack { T v[VEC]; };
+  const int half = rot >> 1, hv = half / VEC, pv = (dim - rot) / VEC, vv = vdim / VEC;
+  const int nq = H * hv, nk = G * hv, np = G * pv, items = nq + nk + np + G * vv;
+  for (int it = threadIdx.x; it < tok_per_cta * items; it += blockDim.x) {
+    const int64_t t = (int64_t)blockIdx.x * tok_per_cta + it / items;
+    if (t >= tokens) return;
+    int i = it % items;
+    T* row = qkv + t * ld;
+    const int pos = token_pos[t];
+    const int64_t crow = i < nq ? 0 : ((int64_t)block_tables[(int64_t)token_seq[t] * max_blocks + pos / block_size] *
+                                           block_size + pos % block_size) * G;
+    if (i < nq + nk) {
+      const int head = i / hv, c = (i % hv) * VEC;            // q heads, then k heads: they sit side by side in the row
+      T* src = row + head * dim + c;
+      T* dst = i < nq ? src : k_cache + (crow + head - H) * dim + c;
+      const Pack a = *reinterpret_cast<const Pack*>(src), b = *reinterpret_cast<const Pack*>(src + half);
+      const float* cs = table + (int64_t)pos * rot + c;
+      float cc[VEC], sn[VEC];
+      load_vec<T, VEC>(cs, true, 0, cc);
+      load_vec<T, VEC>(cs, true, half, sn);
+      Pack oa, ob;
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) {
+        const float u = to_f32<T>(a.v[e]), v = to_f32<T>(b.v[e]);
+        oa.v[e] = from_f32<T>(u * cc[e] - v * sn[e]);
+        ob.v[e] = from_f32<T>(v * cc[e] + u * sn[e]);
+      }
+      *reinterpret_cast<Pack*>(dst) = oa;
+      *reinterpret_cast<Pack*>(dst + half) = ob;
+      continue;
+    }
+    i -= nq + nk;
+    if (i < np) {
+      const int g = i / pv, c = rot + (i % pv) * VEC;
+      *reinterpret_cast<Pack*>(k_cache + (crow + g) * dim + c) = *reinterpret_cast<const Pack*>(row + (H + g) * dim + c);
+    } else {
+      i -= np;
+      *reinterpret_cast<Pack*>(v_cache + crow * vdim + i * VEC) =
+          *reinterpret_cast<const Pack*>(row + (H + G) * dim + i * VEC);
+    }
   }
 }
 
@@ -2427,7 +2638,7 @@ int cb_paged_bias_attention(const void* q, int64_t ldq, const void* k_cache, con
                             const int* token_seq, const int* token_pos, const float* bias_table, const int* bucket_start,
                             int nbuckets, void* out, int64_t tokens, int heads, int kv_heads, int dim, int vdim, int ldv,
                             int block_size, int max_blocks, float scale, int sink, int mask_block, const float* sink_vals,
-                            const float* slopes, int window, int dtype, cudaStream_t st) {
+                            const float* slopes, int window, int keep_first, int dtype, cudaStream_t st) {
   if (tokens == 0) return 0;
   if (vdim > 32 * ATT_MAX_VREG || heads % kv_heads != 0) return (int)cudaErrorInvalidValue;
   const int nwarps = 4;
@@ -2437,20 +2648,20 @@ int cb_paged_bias_attention(const void* q, int64_t ldq, const void* k_cache, con
     paged_bias_attention_kernel<T><<<(unsigned)((units + nwarps - 1) / nwarps), nwarps * 32, smem, st>>>(
         (const T*)q, ldq, (const T*)k_cache, (const T*)v_cache, block_tables, token_seq, token_pos, bias_table,
         bucket_start, nbuckets, (T*)out, tokens, heads, kv_heads, dim, vdim, ldv, block_size, max_blocks, scale, sink,
-        mask_block, sink_vals, slopes, window);
+        mask_block, sink_vals, slopes, window, keep_first);
   });
   return CB_LAUNCH_CHECK();
 }
 
 // 16-bit dtypes, widths that are multiples of 8 and at most 256: the tensor-core kernel.  `chunk` > 0 (a multiple of 64)
-// splits the keys over CTAs; part_o [tokens x heads x max_splits x vdim] and part_ml [.. x 2] are its fp32 workspace.
+// splits the key tile lists over CTAs; part_o [tokens x heads x max_splits x vdim] and part_ml [.. x 2] are its fp32 workspace.
 int cb_paged_bias_attention_mma(const void* q, int64_t ldq, const void* k_cache, const void* v_cache,
                                 const int* block_tables, const int* cu_q, const int* ctx_len, const int* token_pos,
-                                const float* bias_table, const uint8_t* lut, int lut_n, int nbuckets, void* out,
-                                int64_t tokens, int nseq, int max_q, int heads, int kv_heads, int dim, int vdim, int ldv,
+                                const int* token_seq, const float* bias_table, const uint8_t* lut, int lut_n,
+                                int nbuckets, void* out, int64_t tokens, int nseq, int max_q, int heads, int kv_heads, int dim, int vdim, int ldv,
                                 int block_size, int max_blocks, float scale, int sink, int chunk, int max_splits,
                                 float* part_o, float* part_ml, int mask_block, int wide_weights, const float* sink_vals,
-                                const float* slopes, int window, int dtype, cudaStream_t st) {
+                                const float* slopes, int window, int keep_first, int dtype, cudaStream_t st) {
   if (nseq == 0 || max_q == 0) return 0;
   if (heads % kv_heads != 0 || dim % 8 != 0 || vdim % 8 != 0 || dim > 256 || vdim > 256 || (ldq & 7) || ((uintptr_t)q & 15) ||
       (ldv & 7) || ldv < vdim ||
@@ -2459,22 +2670,14 @@ int cb_paged_bias_attention_mma(const void* q, int64_t ldq, const void* k_cache,
   const int dmax = dim > vdim ? dim : vdim;
   const bool wide = max_q * (heads / kv_heads) > 64;      // 128 query rows per CTA (32 per warp) once a portion fills them
   const bool few = max_q * (heads / kv_heads) <= 16;      // decode steps: one m16 tile per sequence, warps split the keys
+#define CB_ATT_ARGS                                                                                                   \
+  q, ldq, k_cache, v_cache, block_tables, cu_q, ctx_len, token_pos, token_seq, bias_table, lut, lut_n, nbuckets, out,  \
+      tokens, nseq, max_q, heads, kv_heads, dim, vdim, ldv, block_size, max_blocks, scale, sink, chunk, max_splits,    \
+      part_o, part_ml, mask_block, wide_weights, sink_vals, slopes, window, keep_first, st
 #define CB_ATT_MMA(T, D)                                                                                              \
-  if (few)                                                                                                            \
-    return launch_attention_mma<T, D, 1, true>(q, ldq, k_cache, v_cache, block_tables, cu_q, ctx_len, token_pos,       \
-                                               bias_table, lut, lut_n, nbuckets, out, tokens, nseq, max_q, heads,      \
-                                               kv_heads, dim, vdim, ldv, block_size, max_blocks, scale, sink, chunk,   \
-                                               max_splits, part_o, part_ml, mask_block, wide_weights, sink_vals,       \
-                                               slopes, window, st);                                                    \
-  if (wide)                                                                                                           \
-    return launch_attention_mma<T, D, 2>(q, ldq, k_cache, v_cache, block_tables, cu_q, ctx_len, token_pos, bias_table, \
-                                         lut, lut_n, nbuckets, out, tokens, nseq, max_q, heads, kv_heads, dim, vdim,  \
-                                         ldv, block_size, max_blocks, scale, sink, chunk, max_splits, part_o, part_ml, \
-                                         mask_block, wide_weights, sink_vals, slopes, window, st);                    \
-  return launch_attention_mma<T, D, 1>(q, ldq, k_cache, v_cache, block_tables, cu_q, ctx_len, token_pos, bias_table,  \
-                                       lut, lut_n, nbuckets, out, tokens, nseq, max_q, heads, kv_heads, dim, vdim,   \
-                                       ldv, block_size, max_blocks, scale, sink, chunk, max_splits, part_o, part_ml,  \
-                                       mask_block, wide_weights, sink_vals, slopes, window, st)
+  if (few) return launch_attention_mma<T, D, 1, true>(CB_ATT_ARGS);                                                   \
+  if (wide) return launch_attention_mma<T, D, 2>(CB_ATT_ARGS);                                                        \
+  return launch_attention_mma<T, D, 1>(CB_ATT_ARGS)
   CB_DISPATCH_HALF(dtype, T, {
     if (dmax <= 32) { CB_ATT_MMA(T, 32); }
     else if (dmax <= 64) { CB_ATT_MMA(T, 64); }
@@ -2482,12 +2685,10 @@ int cb_paged_bias_attention_mma(const void* q, int64_t ldq, const void* k_cache,
     else {                                               // 129..256 wide rows: one m16 tile per warp, one CTA per SM
       // (no key-splitting form here: at this width joining four 16 x 256 accumulators through shared memory costs more
       // than the three idle warps of a short decode CTA, measured 18.9 us against 14.1 us on 8 x 2048 keys)
-      return launch_attention_mma<T, 256, 1>(q, ldq, k_cache, v_cache, block_tables, cu_q, ctx_len, token_pos, bias_table,
-                                             lut, lut_n, nbuckets, out, tokens, nseq, max_q, heads, kv_heads, dim, vdim,
-                                             ldv, block_size, max_blocks, scale, sink, chunk, max_splits, part_o, part_ml,
-                                             mask_block, wide_weights, sink_vals, slopes, window, st);
+      return launch_attention_mma<T, 256, 1>(CB_ATT_ARGS);
     }
   });
+#undef CB_ATT_ARGS
 #undef CB_ATT_MMA
   return CB_LAUNCH_CHECK();
 }
@@ -2577,6 +2778,65 @@ int cb_sigmoid_gate_mul(void* o, const void* gate, int64_t ldg, int64_t tokens, 
     const unsigned grid = (unsigned)((total + 255) / 256 < 148 * 16 ? (total + 255) / 256 : 148 * 16);
     if (vec) sigmoid_gate_mul_kernel<T, V><<<grid, 256, 0, st>>>((T*)o, (const T*)gate, ldg, tokens, C);
     else sigmoid_gate_mul_kernel<T, 1><<<grid, 256, 0, st>>>((T*)o, (const T*)gate, ldg, tokens, C);
+  });
+  return CB_LAUNCH_CHECK();
+}
+
+// x [tokens, W] fp32 += n_o(y) (y itself without n_o; nothing without y); h = n_i(x) when n_i is given.  A norm is absent
+// when its weight pointer is null.  y and h: fp32 or the 16-bit type `dtype`; the norms' parameters alike (p_f32).
+int cb_stream_tanh_norm(float* x, const void* y, int64_t ldy, int y_f32, const void* oa, const void* ow, const void* ob,
+                        const void* ia, const void* iw, const void* ib, int p_f32, void* h, int h_f32, int64_t tokens, int W,
+                        int dtype, cudaStream_t st) {
+  if (tokens == 0 || W == 0) return 0;
+  if (iw != nullptr && h == nullptr) return (int)cudaErrorInvalidValue;
+  const TanhNorm no{oa, ow, ob, p_f32}, ni{ia, iw, ib, p_f32};
+  auto al = [](const void* p) { return ((uintptr_t)p & 15) == 0; };
+  const bool vec = W % 4 == 0 && ldy % 4 == 0 && al(x) && al(y) && al(ow) && al(ob) && al(iw) && al(ib) && al(h);
+  const int cols = vec ? 128 * 4 : 128;
+  const int gx = (W + cols - 1) / cols;
+  int64_t gy = (tokens + TANH_ROWS - 1) / TANH_ROWS;
+  const int64_t cap = (148 * 16 + gx - 1) / gx;
+  if (gy > cap) gy = cap;
+  dim3 grid(gx, (unsigned)gy);
+  CB_DISPATCH_FLOAT(dtype, T, {
+    if (vec) stream_tanh_norm_kernel<T, 4><<<grid, 128, 0, st>>>(x, y, ldy, y_f32, no, ni, h, h_f32, tokens, W);
+    else stream_tanh_norm_kernel<T, 1><<<grid, 128, 0, st>>>(x, y, ldy, y_f32, no, ni, h, h_f32, tokens, W);
+  });
+  return CB_LAUNCH_CHECK();
+}
+
+int cb_router_sigmoid(const float* logits, int64_t ldz, const float* corr, float* w, int64_t* idx, int64_t tokens, int E, int K,
+                      int groups, int keep, int renorm, cudaStream_t st) {
+  if (tokens == 0) return 0;
+  const size_t smem = (size_t)ROUTER_WARPS * (E + groups) * sizeof(float);
+  if (E < 1 || K < 1 || groups < 1 || E % groups != 0 || keep < 1 || keep > groups || K > keep * (E / groups) || smem > 48 * 1024)
+    return (int)cudaErrorInvalidValue;
+  router_sigmoid_kernel<<<(unsigned)((tokens + ROUTER_WARPS - 1) / ROUTER_WARPS), ROUTER_WARPS * 32, smem, st>>>(
+      logits, ldz, corr, w, idx, tokens, E, K, groups, keep, renorm);
+  return CB_LAUNCH_CHECK();
+}
+
+int cb_rotary_kv_write(void* qkv, int64_t ld, int64_t tokens, int H, int G, int dim, int vdim, int rot, const float* table,
+                       void* k_cache, void* v_cache, const int* block_tables, const int* token_seq, const int* token_pos,
+                       int block_size, int max_blocks, int dtype, cudaStream_t st) {
+  if (tokens == 0) return 0;
+  if (rot > dim || (rot & 1) || (rot > 0 && table == nullptr)) return (int)cudaErrorInvalidValue;
+  CB_DISPATCH_FLOAT(dtype, T, {
+    constexpr int V = 16 / sizeof(T);
+    const bool vec = (rot / 2) % V == 0 && dim % V == 0 && vdim % V == 0 && ld % V == 0 && ((uintptr_t)qkv & 15) == 0 &&
+                     ((uintptr_t)k_cache & 15) == 0 && ((uintptr_t)v_cache & 15) == 0 && ((uintptr_t)table & 31) == 0;
+    const int v = vec ? V : 1;
+    const int items = (H * (rot / 2) + G * (rot / 2 + dim - rot) + G * vdim) / v;
+    const int per = items >= 256 ? 1 : 256 / items;
+    const unsigned grid = (unsigned)((tokens + per - 1) / per);
+    if (vec)
+      rotary_kv_write_kernel<T, V><<<grid, 256, 0, st>>>((T*)qkv, ld, tokens, H, G, dim, vdim, rot, table, (T*)k_cache,
+                                                         (T*)v_cache, block_tables, token_seq, token_pos, block_size,
+                                                         max_blocks, per);
+    else
+      rotary_kv_write_kernel<T, 1><<<grid, 256, 0, st>>>((T*)qkv, ld, tokens, H, G, dim, vdim, rot, table, (T*)k_cache,
+                                                         (T*)v_cache, block_tables, token_seq, token_pos, block_size,
+                                                         max_blocks, per);
   });
   return CB_LAUNCH_CHECK();
 }

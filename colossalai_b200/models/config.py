@@ -75,7 +75,9 @@ class MixerSpec:
     activation; its last inputs are carried like a recurrent state); `head_norm` (RMS norm of every q / k head with one
     weight over the head's channels per projection); `values_from_keys` (no value projection: the values are the keys as
     they leave the convolution, before any norm); `dist_slopes` (score minus 2^(-8 (h + 1) / heads) x distance);
-    `window` (a position sees itself and the window - 1 positions before it); `sink_learned` (the sink's score is a
+    `window` (a position sees itself and the window - 1 positions before it), `keep_first` (with a window: the first that
+    many positions of the sequence stay visible at any distance); `rot_scaling`; `bias` (biases in the projection the mixer
+    starts with); `sink_learned` (the sink's score is a
     learned number per head instead of 0)."""
 
     kind: str = "attention"
@@ -113,7 +115,9 @@ class MixerSpec:
     q_rank: int = 0                   # latent: width of the normalised query latent (0 = queries straight from the input)
     window: int = 0                   # attention / latent: > 0 keeps the keys pos - window + 1 .. pos
     sink_learned: bool = False        # the softmax sink's score is a learned number per head (implies a sink)
-    rot_scaling: Optional[List[float]] = None     # (factor, original length, fast, slow): stretched slow frequencies
+    keep_first: int = 0               # attention: keys 0 .. keep_first - 1 stay visible beside the window
+    rot_scaling: Optional[List[float]] = None     # (factor, original length, fast, slow): stretched slow frequencies;
+                                                  # (factor,): every frequency divided by it
     head_norm: bool = False           # attention: RMS norm per q / k head with a weight shared by the heads
     values_from_keys: bool = False    # attention: values = keys before their norm (no value projection)
     dist_slopes: bool = False         # attention: score -= 2^(-8 (h + 1) / heads) * (query position - key position)
@@ -160,12 +164,17 @@ class MixerSpec:
 
 @dataclass
 class ExpertFFSpec:
-    """Routed feed-forward of one layer: `experts` gated experts of width `ff`, every token uses the `top` of largest
-    softmax score (weights renormalised to one), plus an optional shared expert of width `shared_ff` for every token.
-    Expert activation `act`: "clamped": g = min(gate, limit), u = clamp(up, -limit, limit),
-    y = g * sigmoid(alpha * g) * (u + 1); "silu": y = silu(gate) * up.  `shared_gate`: the shared expert's output is
-    multiplied by sigmoid(w_sg . h), one number per token.  (Softmax over all experts renormalised over the chosen ones
-    equals the softmax over the chosen logits alone.)"""
+    """Routed feed-forward of one layer: `experts` experts of width `ff`, every token uses `top` of them, plus an optional
+    shared expert of width `shared_ff` for every token.  Expert activation `act`: "clamped": g = min(gate, limit),
+    u = clamp(up, -limit, limit), y = g * sigmoid(alpha * g) * (u + 1); "silu": y = silu(gate) * up; "relu2" (experts without
+    a gate matrix): y = max(up, 0)^2.  `shared_gate`: the shared expert's output is multiplied by sigmoid(w_sg . h), one
+    number per token.
+
+    `score` "softmax": the `top` experts of largest softmax score, weights renormalised to one (equal to the softmax over
+    the chosen logits alone).  `score` "sigmoid": s = sigmoid(logit); experts are chosen by s (plus a learned number per
+    expert with `correction`) and weighted by s itself, renormalised to one only with `renormalize`; with `groups` > 1 the
+    experts form equal groups of neighbours, a group's score is the sum of its two largest choice scores, and only experts
+    of the `keep_groups` best groups can be chosen."""
 
     experts: int = 1
     top: int = 1
@@ -176,6 +185,18 @@ class ExpertFFSpec:
     shared_limit: float = 7.0
     act: str = "clamped"
     shared_gate: bool = False
+    score: str = "softmax"
+    correction: bool = False
+    renormalize: bool = True
+    groups: int = 1
+    keep_groups: int = 1
+
+    def __post_init__(self) -> None:
+        assert self.act in ("clamped", "silu", "relu2") and self.score in ("softmax", "sigmoid")
+        assert self.act != "relu2" or not self.shared_ff, "shared experts are gated units"
+        assert self.score == "sigmoid" or (self.groups == 1 and not self.correction and self.renormalize)
+        assert self.experts % self.groups == 0 and 1 <= self.keep_groups <= self.groups
+        assert self.top <= self.keep_groups * (self.experts // self.groups), "more choices than experts that can be chosen"
 
 
 @dataclass
@@ -205,7 +226,7 @@ class ModelConfig:
     head_dim: Optional[int] = None
     max_position_embeddings: int = 4096
     norm_eps: float = 1e-5
-    norm_type: str = "rms"            # "rms" | "layer"
+    norm_type: str = "rms"            # "rms" | "layer" | "tanh": tanh(alpha x) w + b element by element (no statistics)
     hidden_act: str = "silu"
     glu: bool = True                  # gated MLP (SwiGLU / GeGLU) vs. plain 2-layer MLP
     attention_bias: bool = False
@@ -241,7 +262,11 @@ class ModelConfig:
     v_head_dim: int = 0
     # hybrid decoders: one spec per layer (mixer kind and sizes, feed-forward width) instead of the uniform fields above
     layer_specs: Optional[List[LayerSpec]] = None
-    norm_placement: str = "pre"       # "pre": sublayer(norm(x)); "sublayer_out": x + residual_mult * norm(sublayer(x))
+    norm_placement: str = "pre"       # "pre": sublayer(norm(x)); "sublayer_out": x + residual_mult * norm(sublayer(x));
+                                      # "both": x + residual_mult * norm'(sublayer(norm(x))), two norms per sublayer
+    # shared layers: the layers (indices into `layer_specs`) in the order they run, when some run more than once with the
+    # same weights; every run has a cache / state of its own.  None: each layer once
+    layer_order: Optional[List[int]] = None
     residual_mult: float = 1.0
     norm_weight_offset: float = 0.0   # zero-centred norm weights: the norm multiplies by (offset + w)
     fp32_residual: bool = False       # the residual stream stays in fp32 whatever the compute dtype
@@ -287,8 +312,12 @@ class ModelConfig:
 
     def layer_runs(self) -> List[Tuple[int, Optional[int]]]:
         """(layer, pass) in execution order; pass is None outside the looped span.  The index into this list is the
-        layer run's cache index: a layer of the span owns one cache / state per pass."""
+        layer run's cache index: a layer of the span (or one that `layer_order` lists several times) owns one cache / state
+        per run."""
         n = self.num_hidden_layers
+        if self.layer_order is not None:
+            assert not self.looped, "a model has either a looped span or an order of layers"
+            return [(i, None) for i in self.layer_order]
         if not self.looped:
             return [(i, None) for i in range(n)]
         a, b = self.loop_start, self.loop_stop

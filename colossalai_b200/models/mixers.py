@@ -17,7 +17,7 @@
 `BiasSinkAttention` also covers plain paged softmax attention with rotary positions (half or interleaved pairs, on a part
 of the head), a weightless unit norm of q / k heads, a block mask (a position sees its own block of positions only), a
 sigmoid output gate, a short convolution on q | k, an RMS norm per q / k head with a shared weight, values taken from the
-keys, a linear distance penalty per head, a sliding window and a learned sink score: every one of these is a field of the
+keys, a linear distance penalty per head, a sliding window (also with the first keys kept) and a learned sink score: every one of these is a field of the
 `MixerSpec`.
 
 Every mixer keeps the call signature of `Attention` (`forward(x, meta, rope, kv_cache)`) and is selected per layer by
@@ -68,6 +68,7 @@ class BiasSinkAttention(_MixerBase):
         assert not spec.values_from_keys or (dv == d and not spec.v_mix), "values taken from the keys are key-wide"
         assert not (spec.conv and (spec.rot_dims or spec.head_unit_norm or spec.proj_norm)), \
             "the convolution on q | k is followed by the per-head norm only"
+        assert not (spec.keep_first and not (spec.window or spec.mask_block)), "kept first keys go with a window"
         # q | k | v (| output gate): one GEMM reads the layer input (no v with `values_from_keys`)
         self.v_width = 0 if spec.values_from_keys else G * dv
         self.qkv_proj = nn.Linear(cfg.hidden_size, H * d + G * d + self.v_width + (H * dv if spec.out_gate else 0),
@@ -110,9 +111,19 @@ class BiasSinkAttention(_MixerBase):
         elif sp.head_norm:
             qk = mops.head_rms_norm(qk if sp.conv else qkv, H, G, d, self.q_head_norm_weight, self.k_head_norm_weight, eps)
             q, k = qk[:, : H * d], qk[:, H * d:]
-        if sp.rot_dims or sp.head_unit_norm:
+        fused_write = not (sp.rot_interleaved or sp.head_unit_norm or sp.proj_norm or sp.v_mix or sp.conv or sp.head_norm
+                           or sp.values_from_keys)
+        if fused_write:
+            # one pass over q | k | v: queries turned in place, keys turned on their way into their pages, values copied
+            kc, vc = kv_cache.pages(self.layer_idx)
+            table = mops.rotary_table(kv_cache.max_len_host, sp.rot_dims, sp.rot_base, x.device, sp.rot_scaling) \
+                if sp.rot_dims else None
+            mops.rotary_kv_write(qkv, H, G, d, dv, sp.rot_dims, table, kc, vc, kv_cache.block_tables, kv_cache.ragged)
+            k = v = None
+        elif sp.rot_dims or sp.head_unit_norm:
             # q and k heads sit side by side in the projection: rotated and normalised in place, in one launch
-            table = mops.rotary_table(kv_cache.max_len_host, sp.rot_dims, sp.rot_base, x.device) if sp.rot_dims else None
+            table = mops.rotary_table(kv_cache.max_len_host, sp.rot_dims, sp.rot_base, x.device, sp.rot_scaling) \
+                if sp.rot_dims else None
             mops.rotary_unit_norm(qkv, H + G, d, sp.rot_dims, sp.rot_interleaved, table, kv_cache.ragged.token_pos,
                                   eps if sp.head_unit_norm else None)
         if sp.proj_norm:
@@ -138,7 +149,7 @@ class BiasSinkAttention(_MixerBase):
         o = kv_cache.attend_ragged(self.layer_idx, q, k, v, self.scale, bias_table=table, bucket_starts=starts,
                                    sink=sp.sink or sp.sink_learned, v_other=v_other, lam=lam, lut=lut,
                                    mask_block=sp.mask_block, wide_weights=sp.wide_weights, sink_values=sinks,
-                                   slopes=slopes, window=sp.window)
+                                   slopes=slopes, window=sp.window, keep_first=sp.keep_first)
         if sp.out_gate:
             o = mops.sigmoid_gate_mul(o, gate)
         return self.o_proj(o)

@@ -12,7 +12,7 @@ Parity: reference `EPMixtralSparseMoeBlock` (`colossalai/shardformer/modeling/mi
 from __future__ import annotations
 
 import math
-from typing import Optional, Tuple
+from typing import Dict, Optional, Tuple
 
 import torch
 import torch.nn as nn
@@ -23,7 +23,7 @@ from ..parallel import comm
 from ..tensor.moe_tensor import set_moe_tensor_ep_group
 from .config import ModelConfig
 
-__all__ = ["SparseMoE", "Router", "GroupedExperts", "ClampedGLU", "ClampedExpertFF"]
+__all__ = ["SparseMoE", "Router", "GroupedExperts", "ClampedGLU", "RoutedExpertFF"]
 
 
 class Router(nn.Module):
@@ -64,14 +64,18 @@ class Router(nn.Module):
 class GroupedExperts(nn.Module):
     """E_local experts stored as batched weights; forward runs on tokens grouped (sorted) by local expert."""
 
-    def __init__(self, cfg: ModelConfig, num_local_experts: int, intermediate: int, gated_act=None) -> None:
+    def __init__(self, cfg: ModelConfig, num_local_experts: int, intermediate: int, gated_act=None,
+                 act: Optional[str] = None) -> None:
         """`gated_act(h, valid_rows)`: a gated activation on the packed gate|up rows that replaces the config's
-        `hidden_act` (the experts are then gated whatever `cfg.glu` says)."""
+        `hidden_act` (the experts are then gated whatever `cfg.glu` says).  `act`: the name of an activation on the up
+        rows alone (the experts then have no gate matrix, whatever `cfg.glu` says)."""
         super().__init__()
         self.cfg, self.num_local_experts, self.intermediate = cfg, num_local_experts, intermediate
         self.gated_act = gated_act
+        self.glu = gated_act is not None or (cfg.glu and act is None)
+        self.act = act or cfg.hidden_act
         H = cfg.hidden_size
-        up_out = 2 * intermediate if (cfg.glu or gated_act is not None) else intermediate
+        up_out = 2 * intermediate if self.glu else intermediate
         self.w_up = nn.Parameter(torch.empty(num_local_experts, up_out, H))      # gate|up fused
         self.w_down = nn.Parameter(torch.empty(num_local_experts, H, intermediate))
         nn.init.normal_(self.w_up, std=cfg.initializer_range)        # (on meta: recorded by the lazy-init log only)
@@ -86,8 +90,7 @@ class GroupedExperts(nn.Module):
             return grouped_linear(self.gated_act(h, counts.sum()), self.w_down, counts)
         # rows past sum(counts) are padding of an over-allocated receive buffer: the activation skips them (the count
         # stays on the device)
-        h = ops.glu(h, self.cfg.hidden_act, valid_rows=counts.sum()) if self.cfg.glu \
-            else ops.get_activation(self.cfg.hidden_act)(h)
+        h = ops.glu(h, self.act, valid_rows=counts.sum()) if self.glu else ops.get_activation(self.act)(h)
         return grouped_linear(h, self.w_down, counts)
 
 
@@ -213,28 +216,38 @@ class SiluGLU(nn.Module):
         return self.down_proj(silu_glu(self.gate_up_proj(x)))
 
 
-class ClampedExpertFF(nn.Module):
+class RoutedExpertFF(nn.Module):
     """Routed feed-forward of a hybrid decoder layer (`LayerSpec.moe`): router scores = softmax over ALL experts in fp32,
-    the `top` largest are used with their scores renormalised to one (+ 1e-20 in the divisor); experts and the optional
-    shared expert are `ClampedGLU`s without biases.  The routed part runs as two grouped GEMMs over the token rows sorted
+    the `top` largest are used with their scores renormalised to one (+ 1e-20 in the divisor) - or, with
+    `spec.score == "sigmoid"`, sigmoid scores with a learned selection correction and group-limited choice
+    (`ops.moe.router_sigmoid_topk`); experts and the optional shared expert are `ClampedGLU`s without biases.  The routed part runs as two grouped GEMMs over the token rows sorted
     by expert and is combined in fp32 by a gather in a fixed order (row j of a token is its j-th choice), so a token's
     result does not depend on what else is in the batch.  `forward` returns (routed sum fp32, shared output or None):
     the caller adds both to the fp32 residual stream.
 
-    `spec.act == "silu"`: the experts are plain `silu(gate) * up` units.  `spec.shared_gate`: the shared expert's output
+    `spec.act == "silu"`: the experts are plain `silu(gate) * up` units; "relu2": max(up, 0)^2, no gate matrix.  `spec.shared_gate`: the shared expert's output
     is multiplied by sigmoid(w_sg . h) per token - w_sg is the router matrix's last row, so the gate's logit comes out of
     the router's fp32 product - and joins the routed rows in the fp32 gather; `forward` then returns that one fp32 sum."""
 
     def __init__(self, cfg: ModelConfig, spec) -> None:
         super().__init__()
         self.cfg, self.spec = cfg, spec
-        assert spec.act in ("clamped", "silu") and not (spec.shared_gate and not spec.shared_ff)
+        assert not (spec.shared_gate and not spec.shared_ff)
         self.router = nn.Linear(cfg.hidden_size, spec.experts + int(spec.shared_gate), bias=False)
-        self.experts = GroupedExperts(cfg, spec.experts, spec.ff, gated_act=self._act)
+        self.experts = GroupedExperts(cfg, spec.experts, spec.ff, act=spec.act) if spec.act == "relu2" else \
+            GroupedExperts(cfg, spec.experts, spec.ff, gated_act=self._act)
+        if spec.correction:
+            self.correction = nn.Parameter(torch.zeros(spec.experts))
+            self._correction32: Dict[str, torch.Tensor] = {}
         if spec.shared_ff:
             self.shared = SiluGLU(cfg, spec.shared_ff) if spec.act == "silu" else \
                 ClampedGLU(cfg, spec.shared_ff, spec.shared_limit, spec.alpha)
         self.shard_config = None
+
+    def _apply(self, fn, *a, **k):          # parameters moved or cast: the fp32 copy of the correction is rebuilt
+        if self.spec.correction:
+            self._correction32 = {}
+        return super()._apply(fn, *a, **k)
 
     def _act(self, h: torch.Tensor, valid_rows) -> torch.Tensor:
         if self.spec.act == "silu":
@@ -256,6 +269,17 @@ class ClampedExpertFF(nn.Module):
         sg = None
         if self.spec.shared_gate:
             logits, sg = logits[:, : self.spec.experts], logits[:, self.spec.experts]
+        if self.spec.score == "sigmoid":
+            from ..ops.moe import router_sigmoid_topk
+
+            corr = None
+            if self.spec.correction:
+                key = str(x.device)
+                if key not in self._correction32:
+                    self._correction32[key] = self.correction.detach().float().contiguous()
+                corr = self._correction32[key]
+            return router_sigmoid_topk(logits, self.spec.top, corr, self.spec.groups, self.spec.keep_groups,
+                                       self.spec.renormalize) + (sg,)
         if x.dtype == torch.float32:            # 32-bit serving: IEEE exponentials
             p = torch.softmax(logits, -1)
             w, idx = torch.topk(p, self.spec.top, dim=-1)

@@ -33,7 +33,7 @@ from ..shardformer.layer._operation import (
 )
 from ..shardformer.layer.attn import RingAttention
 from ..shardformer.layer.loss import dist_cross_entropy
-from ..shardformer.layer.normalization import FusedLayerNorm, FusedRMSNorm
+from ..shardformer.layer.normalization import DynamicTanh, FusedLayerNorm, FusedRMSNorm
 from .config import ModelConfig
 
 __all__ = ["SeqMeta", "Attention", "MLP", "DecoderLayer", "TransformerModel", "TransformerLMHeadModel",
@@ -56,6 +56,7 @@ class SeqMeta:
     pending: Optional[list] = None              # fp32 stream: sublayer outputs not added yet (the next norm's kernel
                                                 # adds them) and a [W] vector added to every token (`pending_row`)
     pending_row: Optional[torch.Tensor] = None
+    pending_norm: Optional[nn.Module] = None    # norm that the (single) pending output passes before it is added
     history: Optional[tuple] = None             # depth average: (stream history, terms, their weights, where the sum goes,
                                                 # whether its compute-dtype copy is wanted) for the layer's last sublayer
 
@@ -77,7 +78,33 @@ def build_norm(cfg: ModelConfig, hidden: Optional[int] = None) -> nn.Module:
         norm = FusedRMSNorm(h, eps=cfg.norm_eps, offset=cfg.norm_weight_offset)
         norm.reset_parameters()
         return norm
+    if cfg.norm_type == "tanh":
+        return DynamicTanh(h)
     return FusedLayerNorm(h, eps=cfg.norm_eps, bias=cfg.norm_bias)
+
+
+def advance_stream(x: torch.Tensor, meta: SeqMeta, norm: Optional[nn.Module], cfg: ModelConfig) -> Optional[torch.Tensor]:
+    """The fp32 stream between two sublayers: adds what is pending (`meta.pending`, passed through `meta.pending_norm` where a
+    sublayer's output is normalised; `meta.pending_row`) to x in place and, with `norm`, returns the new x normalised in the
+    parameters' dtype.  One kernel, except for an output norm that needs the row's statistics (a kernel of its own)."""
+    pend, out_norm, row = meta.pending or (), meta.pending_norm, meta.pending_row
+    meta.pending = meta.pending_norm = meta.pending_row = None
+    if cfg.norm_type == "tanh":
+        assert cfg.residual_mult == 1.0 and row is None and len(pend) <= 1, "elementwise norms take one sublayer output"
+        return ops.mixers.stream_tanh_norm(x, pend[0] if pend else None, None if out_norm is None else out_norm.params,
+                                           None if norm is None else norm.params)
+    if out_norm is not None:
+        assert cfg.norm_type == "rms" and len(pend) == 1
+        ops.rms_norm_residual(x, pend[0], out_norm.weight, cfg.norm_eps, mult=cfg.residual_mult,
+                              offset=cfg.norm_weight_offset, want_cast=False)
+        pend = ()
+    if norm is None:
+        if pend or row is not None:
+            ops.mixers.stream_add_norm(x, pend, row=row)
+        return None
+    assert getattr(norm, "bias", None) is None, "the stream's fused norm carries a weight only"
+    return ops.mixers.stream_add_norm(x, pend, row=row, weight=norm.weight, eps=cfg.norm_eps, kind=cfg.norm_type,
+                                      offset=cfg.norm_weight_offset)
 
 
 def _sc(module: nn.Module):
@@ -371,11 +398,16 @@ class DecoderLayer(nn.Module):
             self.self_attn = MLAttention(cfg, layer_idx) if cfg.use_mla else Attention(cfg, layer_idx)
         if not cfg.parallel_block and (spec is None or spec.ff is not None or spec.moe is not None):
             self.post_attention_layernorm = build_norm(cfg)
+        if cfg.norm_placement == "both":          # norms of the sublayers' outputs beside those of their inputs
+            assert cfg.fp32_residual and not cfg.parallel_block, "norms on both sides of a sublayer run on an fp32 stream"
+            self.mixer_out_norm = build_norm(cfg)
+            if hasattr(self, "post_attention_layernorm"):
+                self.mlp_out_norm = build_norm(cfg)
         moe = cfg.moe
         if spec is not None and spec.moe is not None:
-            from .moe import ClampedExpertFF
+            from .moe import RoutedExpertFF
 
-            self.mlp = ClampedExpertFF(cfg, spec.moe)
+            self.mlp = RoutedExpertFF(cfg, spec.moe)
         elif spec is not None:
             self.mlp = MLP(cfg, spec.ff, act=spec.ff_act) if spec.ff is not None else None
         elif moe is not None and layer_idx >= moe.first_k_dense_replace and (layer_idx % moe.moe_layer_freq == 0):
@@ -429,11 +461,7 @@ class DecoderLayer(nn.Module):
         """Parallel block on an fp32 stream: h = norm(x); x <- x + (mixer(h) + ff(h)).  The sum is left PENDING
         (`meta.pending`): the kernel that normalises the stream for the next layer (or the final norm) first adds the
         pending outputs, in fp32, in one pass over x."""
-        cfg = self.cfg
-        norm = self.input_layernorm
-        h = ops.mixers.stream_add_norm(x, meta.pending or (), row=meta.pending_row, weight=norm.weight, eps=cfg.norm_eps,
-                                       kind=cfg.norm_type, offset=cfg.norm_weight_offset)
-        meta.pending_row = None
+        h = advance_stream(x, meta, self.input_layernorm, self.cfg)
         outs = [self.self_attn(h, meta, rope, kv_cache)]
         if self.mlp is not None:
             y = self.mlp(h)
@@ -442,19 +470,20 @@ class DecoderLayer(nn.Module):
         return x
 
     def _forward_pre_stream(self, x: torch.Tensor, meta: SeqMeta, rope, kv_cache) -> torch.Tensor:
-        """Pre-norm sublayers on an fp32 stream: x <- x + mixer(norm1(x)); x <- x + ff(norm2(x)).  Each sublayer's output
-        is left PENDING and added, in fp32, by the kernel that normalises the stream for the next sublayer (this
+        """Pre-norm sublayers on an fp32 stream: x <- x + mixer(norm1(x)); x <- x + ff(norm2(x)) - with norms on both sides,
+        x <- x + out_norm(mixer(norm1(x))) and so on.  Each sublayer's output is left PENDING and added, in fp32, by the kernel that normalises the stream for the next sublayer (this
         layer's second norm, the next layer's first one, or the final norm): one pass over x per sublayer."""
-        cfg = self.cfg
-        assert getattr(self.input_layernorm, "bias", None) is None, "the stream's fused norm carries a weight only"
-        kw = dict(eps=cfg.norm_eps, kind=cfg.norm_type, offset=cfg.norm_weight_offset)
-        h = ops.mixers.stream_add_norm(x, meta.pending or (), row=meta.pending_row, weight=self.input_layernorm.weight, **kw)
-        meta.pending_row = None
+        both = self.cfg.norm_placement == "both"
+        h = advance_stream(x, meta, self.input_layernorm, self.cfg)
         meta.pending = [self.self_attn(h, meta, rope, kv_cache)]
+        meta.pending_norm = self.mixer_out_norm if both else None
         if self.mlp is not None:
-            h = ops.mixers.stream_add_norm(x, meta.pending, weight=self.post_attention_layernorm.weight, **kw)
+            h = advance_stream(x, meta, self.post_attention_layernorm, self.cfg)
             y = self.mlp(h)
-            meta.pending = [t for t in (y if isinstance(y, tuple) else (y,)) if t is not None]
+            outs = [t for t in (y if isinstance(y, tuple) else (y,)) if t is not None]
+            if both and len(outs) > 1:                     # the output norm reads the sum of the parts
+                outs = [sum(t.float() for t in outs)]
+            meta.pending, meta.pending_norm = outs, (self.mlp_out_norm if both else None)
         return x
 
     def _forward_sublayer_out(self, x: torch.Tensor, meta: SeqMeta, rope, kv_cache) -> torch.Tensor:
@@ -665,14 +694,15 @@ class TransformerModel(nn.Module):
                                               else self.embed_tokens.weight.dtype)
         start, end = self.layer_range()
         n_ckpt = self._num_ckpt_layers(end - start) if self.training else 0
-        stream = cfg.fp32_residual and cfg.norm_placement == "pre" and not cfg.post_norm
+        stream = cfg.fp32_residual and cfg.norm_placement in ("pre", "both") and not cfg.post_norm
         if cfg.depth_average:
             assert sm is None and not cfg.looped, "depth-averaged streams are not split over pipeline stages or looped"
             return self._forward_depth_average(x, meta, rope, kv_cache)
-        if cfg.looped or stream:
+        if cfg.looped or cfg.layer_order is not None or stream:
             # a span of layers may run several times with the same weights: every layer RUN has its own cache / state
             # (the runtime is told which), and every pass starts by adding the embedding output (not the first) and the
-            # pass's learned vector to the stream
+            # pass's learned vector to the stream.  Layers that `layer_order` lists several times run in the
+            # same way, without those additions
             assert sm is None, "looped spans / pending-sum streams are not split over pipeline stages"
             x0 = x
             if cfg.looped:
@@ -690,16 +720,11 @@ class TransformerModel(nn.Module):
                 x = self.layers[i](x, meta, rope, kv_cache)
                 if self.stream_trace is not None:
                     if meta.pending:
-                        ops.mixers.stream_add_norm(x, meta.pending)
-                        meta.pending = None
+                        advance_stream(x, meta, None, cfg)
                     self.stream_trace.append(x.detach().float().clone())
             if stream:
-                pend, meta.pending = meta.pending or (), None
-                if cfg.final_norm:
-                    return ops.mixers.stream_add_norm(x, pend, weight=self.norm.weight, eps=cfg.norm_eps,
-                                                      kind=cfg.norm_type, offset=cfg.norm_weight_offset)
-                ops.mixers.stream_add_norm(x, pend)
-                return x
+                h = advance_stream(x, meta, self.norm if cfg.final_norm else None, cfg)
+                return x if h is None else h
         else:
             for i in range(start, end):
                 layer = self.layers[i]

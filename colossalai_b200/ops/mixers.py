@@ -3,7 +3,8 @@ recurrent state scans (decayed outer-product state with optional rotary position
 outer-product state for selective state spaces and the exponentially gated matrix memory, per-channel gated linear
 recurrence), group RMS norm with a sigmoid / silu gate before or after the norm, rotary positions + unit norm of q / k
 heads, the mean of RMS-normed mixer outputs, RMS norm of a sublayer's output added to an fp32 residual stream, sums into the fp32 stream
-fused with the next RMS / layer norm, rotary positions from an fp32 angle table, the cache rows of latent attention, and
+fused with the next RMS / layer norm or with elementwise tanh norms on both sides of the sum, rotary positions from an
+fp32 angle table (alone, or in one pass with the write of the key / value pages), the cache rows of latent attention, and
 paged attention with a distance-bucket bias and a softmax sink (values optionally read from the key rows).
 
 All ops take a RAGGED step (`RaggedMeta`): for every live sequence its next tokens, how many tokens earlier steps
@@ -28,7 +29,7 @@ __all__ = ["RaggedMeta", "short_conv_silu", "state_scan_decay", "state_scan_delt
            "rms_norm_residual", "rms_norm_f32in", "paged_kv_write_mix", "paged_bias_attention", "log_bucket_starts",
            "bucket_lut", "rotary_table", "rotary_half", "stream_add_norm", "latent_kv_write", "state_scan_ssd",
            "state_scan_mlstm", "lru_scan", "rotary_unit_norm", "sigmoid_gate_mul", "norm_mean", "depth_mix", "poly_norm",
-           "head_rms_norm", "distance_slopes"]
+           "head_rms_norm", "distance_slopes", "stream_tanh_norm", "rotary_kv_write"]
 
 _lib = None
 _SPLIT_BELOW_TILES = 148        # attention steps with fewer CTAs than SMs split their keys
@@ -159,7 +160,8 @@ _rotary_tables = {}
 
 
 def rotary_frequencies(dims: int, base: float, scaling: Optional[Sequence[float]] = None):
-    """(f [dims / 2] float64, factor on cos / sin).  f_i = base^(-2 i / dims).  `scaling` = (s, n, fast, slow) stretches
+    """(f [dims / 2] float64, factor on cos / sin).  f_i = base^(-2 i / dims).  `scaling` = (s,) divides every frequency by
+    s (positions are interpolated linearly; cos and sin stay as they are).  `scaling` = (s, n, fast, slow) stretches
     the slow frequencies for contexts beyond the n positions the model was trained on: with
     d(t) = dims ln(n / (2 pi t)) / (2 ln base) - the channel that turns t times over n positions - lo = max(floor(d(fast)), 0),
     hi = min(ceil(d(slow)), dims - 1) and r_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1), the frequency becomes
@@ -167,6 +169,8 @@ def rotary_frequencies(dims: int, base: float, scaling: Optional[Sequence[float]
     f = torch.tensor(float(base), dtype=torch.float64) ** (-torch.arange(0, dims, 2, dtype=torch.float64) / dims)
     if not scaling:
         return f, 1.0
+    if len(scaling) == 1:
+        return f / float(scaling[0]), 1.0
     s, n, fast, slow = [float(v) for v in scaling]
     d = lambda t: dims * math.log(n / (2.0 * math.pi * t)) / (2.0 * math.log(base))
     lo = max(math.floor(d(fast)), 0)
@@ -749,6 +753,32 @@ def rotary_unit_norm(x: torch.Tensor, heads: int, dim: int, rot_dims: int, inter
     x[:, : heads * dim] = y.reshape(T, heads * dim).to(x.dtype)
 
 
+def rotary_kv_write(qkv: torch.Tensor, heads: int, kv_heads: int, dim: int, vdim: int, rot_dims: int,
+                    table: Optional[torch.Tensor], k_cache: torch.Tensor, v_cache: torch.Tensor,
+                    block_tables: torch.Tensor, meta: RaggedMeta) -> None:
+    """One pass over projection rows q | k | v [T, >= heads x dim + kv_heads x (dim + vdim)] (unit stride inside a row):
+    the first `rot_dims` channels of every q and k head are turned by the token's position (rotate-half pairs, `table` =
+    `rotary_table` of `rot_dims`; fp32 arithmetic, one rounding), the queries in place, the keys on their way into the
+    tokens' rows of `k_cache` [blocks, block_size, kv_heads, dim]; the values go into `v_cache` [.., kv_heads, vdim]."""
+    T = qkv.shape[0]
+    bs = k_cache.shape[1]
+    assert k_cache.shape[2:] == (kv_heads, dim) and v_cache.shape[2:] == (kv_heads, vdim)
+    if use_native(qkv):
+        assert qkv.stride(1) == 1 and k_cache.dtype == qkv.dtype and v_cache.dtype == qkv.dtype
+        assert k_cache.is_contiguous() and v_cache.is_contiguous()
+        assert rot_dims == 0 or (table.dtype == torch.float32 and table.shape[1] == rot_dims)
+        loader.check(_get_lib().cb_rotary_kv_write(
+            loader.ptr(qkv), _i64(qkv.stride(0)), _i64(T), heads, kv_heads, dim, vdim, rot_dims,
+            loader.ptr(table if rot_dims else None), loader.ptr(k_cache), loader.ptr(v_cache), loader.ptr(block_tables),
+            loader.ptr(meta.token_seq), loader.ptr(meta.token_pos), bs, block_tables.shape[1], code(qkv.dtype),
+            loader.stream_ptr()), "rotary_kv_write")
+        loader.launch_counter.add("rotary_kv_write")
+        return
+    rotary_unit_norm(qkv, heads + kv_heads, dim, rot_dims, False, table, meta.token_pos, None)
+    a, b = heads * dim, (heads + kv_heads) * dim
+    paged_kv_write_mix(qkv[:, a:b], qkv[:, b:b + kv_heads * vdim], k_cache, v_cache, block_tables, meta)
+
+
 _NORM_KINDS = {None: 0, "none": 0, "rms": 1, "layer": 2}
 
 
@@ -796,6 +826,41 @@ def stream_add_norm(x: torch.Tensor, addends: Sequence[torch.Tensor] = (), row: 
         d = x - x.mean(-1, keepdim=True)
         y = d / torch.sqrt((d * d).mean(-1, keepdim=True) + eps)
     return (y * (offset + weight.float())).to(out_dtype)
+
+
+def tanh_norm(x: torch.Tensor, alpha: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor) -> torch.Tensor:
+    """tanh(alpha x) * weight + bias element by element in fp32 (PyTorch form)."""
+    return torch.tanh(alpha.float() * x.float()) * weight.float() + bias.float()
+
+
+def stream_tanh_norm(x: torch.Tensor, y: Optional[torch.Tensor] = None, out_norm: Optional[tuple] = None,
+                     in_norm: Optional[tuple] = None) -> Optional[torch.Tensor]:
+    """The fp32 residual stream x [T, W], updated in place, between two sublayers: x += n_o(y) for the output y [T, W]
+    (compute dtype or fp32) of the sublayer before, then h = n_i(x) for the one behind, returned in the parameters' dtype.
+    A norm is a triple (alpha scalar, weight [W], bias [W]): n(z) = tanh(alpha z) * weight + bias, which needs nothing of
+    the rest of the row, so one elementwise kernel does it all.  Without `out_norm` y is added as it is, without y the
+    stream stays, without `in_norm` nothing is returned."""
+    T, W = x.shape
+    assert x.dtype == torch.float32 and (out_norm is None or y is not None)
+    norm = in_norm or out_norm
+    if use_native(x):
+        assert x.is_contiguous() and (y is None or (y.stride(1) == 1 and y.shape == x.shape))
+        dt = norm[1].dtype if norm is not None else (y.dtype if y is not None else torch.float32)
+        assert y is None or y.dtype in (dt, torch.float32)
+        for n in (out_norm, in_norm):
+            assert n is None or all(t.dtype == dt and t.is_contiguous() for t in n)
+        h = torch.empty(T, W, dtype=dt, device=x.device) if in_norm is not None else None
+        f32 = int(dt == torch.float32)
+        pp = lambda n: (None, None, None) if n is None else tuple(loader.ptr(t) for t in n)
+        loader.check(_get_lib().cb_stream_tanh_norm(
+            loader.ptr(x), loader.ptr(y), _i64(0 if y is None else y.stride(0)),
+            int(y is not None and y.dtype == torch.float32), *pp(out_norm), *pp(in_norm), f32, loader.ptr(h), f32, _i64(T),
+            W, code(dt), loader.stream_ptr()), "stream_tanh_norm")
+        loader.launch_counter.add("stream_tanh_norm")
+        return h
+    if y is not None:
+        x += tanh_norm(y, *out_norm) if out_norm is not None else y.float()
+    return None if in_norm is None else tanh_norm(x, *in_norm).to(in_norm[1].dtype)
 
 
 # ------------------------------------------------------------------------------------------------ paged attention
@@ -850,13 +915,23 @@ def paged_kv_write_mix(k: torch.Tensor, v: torch.Tensor, k_cache: torch.Tensor, 
     v_cache.view(v_cache.shape[0], bs, vw)[blk, off] = v
 
 
+def _key_tiles(max_len: int, max_q: int, rep: int, mask_block: int, window: int, keep_first: int) -> int:
+    """Most 64-key tiles that a row tile of the tensor-core kernel can walk: all up to `max_len`; with a window or a block
+    mask those that reach from its first row's first key (rounded down to a tile) to its last row's position, plus the
+    tiles of the kept first keys.  `rep` query heads share a key head; a row tile holds up to 128 rows."""
+    whole = -(-max_len // 64)
+    bound = min(mask_block or max_len, window or max_len)
+    span = bound + min(max_q, 127 // rep + 2) - 1
+    return min(whole, (span + 126) // 64 + -(-keep_first // 64))
+
+
 def paged_bias_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, block_tables: torch.Tensor,
                          meta: RaggedMeta, scale: float, bias_table: Optional[torch.Tensor] = None,
                          bucket_starts: Optional[torch.Tensor] = None, sink: bool = False,
                          lut: Optional[torch.Tensor] = None, tensor_cores: Optional[bool] = None,
                          vdim: Optional[int] = None, mask_block: int = 0, wide_weights: bool = False,
                          sink_values: Optional[torch.Tensor] = None, slopes: Optional[torch.Tensor] = None,
-                         window: int = 0) -> torch.Tensor:
+                         window: int = 0, keep_first: int = 0) -> torch.Tensor:
     """Causal attention of every step token over positions 0..pos of its sequence in the paged cache; with `mask_block`
     only over the positions of its own block, floor(pos / mask_block) * mask_block .. pos (blocks are counted from the
     start of the sequence, whatever the step's cut).
@@ -866,7 +941,8 @@ def paged_bias_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.
     the bucket of the distance (`bucket_starts` [buckets] int32: smallest distance of each bucket); `sink` adds a key of
     score 0 without a value to the softmax - with `sink_values` [heads] fp32 a key of that (unscaled) score per head.
     `slopes` [heads] fp32 takes slope * (pos - key position) off every score; `window` > 0 keeps only the keys
-    pos - window + 1 .. pos.  Returns [T, heads x vdim].
+    pos - window + 1 .. pos and the first `keep_first` keys of the sequence (at their true positions, whatever the window or
+    block mask says).  Returns [T, heads x vdim].
 
     Two kernels: 16-bit inputs whose head widths are multiples of 8 up to 256 run on tensor cores (`lut` = `bucket_lut`
     of the same buckets; built here when absent); everything else - fp32 above all - takes the exact CUDA-core kernel.
@@ -894,36 +970,27 @@ def paged_bias_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.
                                  "that are multiples of 8 up to 256")
             if nb and lut is None:
                 lut = bucket_lut(bucket_starts.tolist()).to(q.device)
-            # few CTAs (decode steps): split the keys so that about two waves of CTAs run, join the parts afterwards
+            # few CTAs (decode steps): split the key tile lists so that about two waves of CTAs run, join the parts
+            # afterwards
             R = heads // G
             tiles = meta.nseq * G * ((meta.max_q * R + 63) // 64)
-            max_len = max(c + n for c, n in zip(meta.ctx_lens, meta.q_lens))
-            if mask_block:
-                max_len = min(max_len, mask_block + 64)       # keys a tile can see: the split is sized for those
-            if window:
-                max_len = min(max_len, window + 64)
+            key_tiles = _key_tiles(max(c + n for c, n in zip(meta.ctx_lens, meta.q_lens)), meta.max_q, R, mask_block, window,
+                                   keep_first)
             chunk = splits = 0
             part_o = part_ml = None
-            if tiles < _SPLIT_BELOW_TILES and max_len >= 256:
-                chunk = max(128, -(-(max_len * tiles // (2 * _SPLIT_BELOW_TILES)) // 64) * 64)
-                splits = -(-max_len // chunk)
-                if splits > 1:
+            if tiles < _SPLIT_BELOW_TILES and key_tiles >= 4:
+                per = max(2, -(-key_tiles * tiles // (2 * _SPLIT_BELOW_TILES)))       # tiles of a chunk
+                if key_tiles > per:
+                    chunk, splits = 64 * per, -(-key_tiles // per)
                     part_o = _workspace("attn_o", T * heads * splits * vdim, q.device)
                     part_ml = _workspace("attn_ml", T * heads * splits * 2, q.device)
-                else:
-                    chunk = splits = 0
-            if (mask_block or window) and splits:
-                max_len = max(c + n for c, n in zip(meta.ctx_lens, meta.q_lens))
-                splits = -(-max_len // chunk)                 # chunks are counted from key 0
-                part_o = _workspace("attn_o", T * heads * splits * vdim, q.device)
-                part_ml = _workspace("attn_ml", T * heads * splits * 2, q.device)
             loader.check(_get_lib().cb_paged_bias_attention_mma(
                 loader.ptr(q), _i64(q.stride(0)), loader.ptr(k_cache), loader.ptr(v_cache), loader.ptr(block_tables),
-                loader.ptr(meta.cu_q), loader.ptr(meta.ctx_len), loader.ptr(meta.token_pos), loader.ptr(bias_table),
-                loader.ptr(lut), 0 if lut is None else lut.numel(), nb, loader.ptr(out), _i64(T), meta.nseq, meta.max_q,
+                loader.ptr(meta.cu_q), loader.ptr(meta.ctx_len), loader.ptr(meta.token_pos), loader.ptr(meta.token_seq),
+                loader.ptr(bias_table), loader.ptr(lut), 0 if lut is None else lut.numel(), nb, loader.ptr(out), _i64(T), meta.nseq, meta.max_q,
                 heads, G, dim, vdim, ldv, bs, block_tables.shape[1], _f(scale), int(sink), chunk, splits,
                 loader.ptr(part_o), loader.ptr(part_ml), int(mask_block), int(wide_weights), loader.ptr(sink_values),
-                loader.ptr(slopes), int(window), code(q.dtype), loader.stream_ptr()),
+                loader.ptr(slopes), int(window), int(keep_first), code(q.dtype), loader.stream_ptr()),
                 "paged_bias_attention_mma")
             loader.launch_counter.add("paged_bias_attention_mma")
             return out
@@ -931,7 +998,7 @@ def paged_bias_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.
             loader.ptr(q), _i64(q.stride(0)), loader.ptr(k_cache), loader.ptr(v_cache), loader.ptr(block_tables),
             loader.ptr(meta.token_seq), loader.ptr(meta.token_pos), loader.ptr(bias_table), loader.ptr(bucket_starts), nb,
             loader.ptr(out), _i64(T), heads, G, dim, vdim, ldv, bs, block_tables.shape[1], _f(scale), int(sink),
-            int(mask_block), loader.ptr(sink_values), loader.ptr(slopes), int(window), code(q.dtype),
+            int(mask_block), loader.ptr(sink_values), loader.ptr(slopes), int(window), int(keep_first), code(q.dtype),
             loader.stream_ptr()), "paged_bias_attention")
         loader.launch_counter.add("paged_bias_attention")
         return out
@@ -951,12 +1018,13 @@ def paged_bias_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.
         if bias_table is not None:
             b = torch.bucketize(dist.clamp(min=0), bucket_starts.to(torch.int64), right=True) - 1
             s = s + bias_table.float()[b].permute(2, 0, 1)
-        s = s.masked_fill(dist[None] < 0, float("-inf"))
+        near = torch.ones_like(dist, dtype=torch.bool)
         if mask_block:
-            same = (torch.arange(c, L)[:, None] // mask_block) == (torch.arange(L)[None, :] // mask_block)
-            s = s.masked_fill(~same[None], float("-inf"))
+            near &= (torch.arange(c, L)[:, None] // mask_block) == (torch.arange(L)[None, :] // mask_block)
         if window:
-            s = s.masked_fill(dist[None] >= window, float("-inf"))
+            near &= dist < window
+        near |= torch.arange(L)[None, :] < keep_first
+        s = s.masked_fill(~(near & (dist >= 0))[None], float("-inf"))
         if slopes is not None:
             s = s - slopes.float()[:, None, None] * dist.clamp(min=0)[None].float()
         if sink:

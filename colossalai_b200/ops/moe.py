@@ -2,7 +2,7 @@
 
  * capacity-based dispatch/combine + cumsum (legacy MoE layer; reference `MoeDispatch`/`MoeCombine`/`moe_cumsum` in
    colossalai/moe/_operation.py:220-330 backed by moe_kernel.cu)
- * fused router softmax + top-k
+ * fused router softmax + top-k; sigmoid router with a selection correction and group-limited top-k
 """
 from __future__ import annotations
 
@@ -151,6 +151,40 @@ def router_topk(logits: torch.Tensor, k: int, renormalize: bool = True, return_p
     if renormalize:
         w = w / w.sum(-1, keepdim=True).clamp_min(1e-20)
     return (w, idx, probs) if return_probs else (w, idx)
+
+
+def router_sigmoid_topk(logits: torch.Tensor, k: int, correction: Optional[torch.Tensor] = None, groups: int = 1,
+                        keep_groups: int = 1, renormalize: bool = False) -> Tuple[torch.Tensor, torch.Tensor]:
+    """fp32 router logits [T, E] -> (weights fp32 [T, k], experts int64 [T, k], in the order of their choice scores).  With
+    s = sigmoid(logits) and choice scores s + correction [E]: the experts form `groups` equal groups of neighbours, a
+    group's score is the sum of its two largest choice scores, experts outside the `keep_groups` best groups cannot be
+    chosen (their choice scores count as minus infinity), the k largest choice scores win and the weights are s itself
+    (`renormalize`: divided by their sum).  IEEE exponentials.  Forward only."""
+    T, E = logits.shape
+    assert E % groups == 0 and 1 <= keep_groups <= groups and k <= keep_groups * (E // groups)
+    if use_native(logits):
+        from .mixers import _get_lib as _mixers_lib
+
+        assert logits.dtype == torch.float32 and logits.stride(1) == 1
+        assert correction is None or (correction.dtype == torch.float32 and correction.is_contiguous())
+        w = torch.empty(T, k, dtype=torch.float32, device=logits.device)
+        idx = torch.empty(T, k, dtype=torch.int64, device=logits.device)
+        loader.check(_mixers_lib().cb_router_sigmoid(
+            loader.ptr(logits), ctypes.c_int64(logits.stride(0)), loader.ptr(correction), loader.ptr(w), loader.ptr(idx),
+            ctypes.c_int64(T), E, k, groups, keep_groups, int(renormalize), loader.stream_ptr()), "router_sigmoid")
+        loader.launch_counter.add("router_sigmoid")
+        return w, idx
+    s = torch.sigmoid(logits.float())
+    c = s if correction is None else s + correction.float()
+    if keep_groups < groups:
+        g = c.view(T, groups, E // groups)
+        score = torch.topk(g, min(2, E // groups), dim=-1).values.sum(-1)
+        best = torch.topk(score, keep_groups, dim=-1).indices
+        keep = torch.zeros(T, groups, dtype=torch.bool, device=c.device).scatter_(1, best, True)
+        c = g.masked_fill(~keep[..., None], float("-inf")).reshape(T, E)
+    idx = torch.topk(c, k, dim=-1).indices
+    w = s.gather(1, idx)
+    return (w / w.sum(-1, keepdim=True).clamp_min(1e-20) if renormalize else w), idx
 
 
 def gather_combine(rows: torch.Tensor, row_of: torch.Tensor, weights: torch.Tensor,

@@ -13,7 +13,7 @@ import torch.nn as nn
 from ... import ops
 from .utils import SeqParallelUtils
 
-__all__ = ["RMSNorm", "LayerNorm", "FusedRMSNorm", "FusedLayerNorm", "BaseLayerNorm"]
+__all__ = ["RMSNorm", "LayerNorm", "FusedRMSNorm", "FusedLayerNorm", "DynamicTanh", "BaseLayerNorm"]
 
 
 class BaseLayerNorm(nn.Module):
@@ -59,6 +59,34 @@ class FusedRMSNorm(BaseLayerNorm):
 
     def extra_repr(self) -> str:
         return f"{self.hidden_size}, eps={self.eps}"
+
+
+class DynamicTanh(BaseLayerNorm):
+    """tanh(alpha x) * weight + bias, element by element in fp32: a norm that computes no mean or variance.  `params` is the
+    triple that `ops.mixers.stream_tanh_norm` fuses into the residual stream's update."""
+
+    def __init__(self, hidden_size: int, alpha: float = 0.5, dtype=None, device=None) -> None:
+        super().__init__()
+        self.init_alpha = alpha
+        self.weight = nn.Parameter(torch.ones(hidden_size, dtype=dtype, device=device))
+        self.bias = nn.Parameter(torch.zeros(hidden_size, dtype=dtype, device=device))
+        self.alpha = nn.Parameter(torch.tensor(float(alpha), dtype=dtype or torch.float32, device=device))
+        self.hidden_size = hidden_size
+
+    def reset_parameters(self) -> None:
+        nn.init.ones_(self.weight)
+        nn.init.zeros_(self.bias)
+        nn.init.constant_(self.alpha, self.init_alpha)
+
+    @property
+    def params(self):
+        return self.alpha, self.weight, self.bias
+
+    def forward(self, x: torch.Tensor) -> torch.Tensor:
+        return ops.mixers.tanh_norm(x, *self.params).to(x.dtype)
+
+    def extra_repr(self) -> str:
+        return f"{self.hidden_size}"
 
 
 class FusedLayerNorm(BaseLayerNorm):

@@ -248,12 +248,12 @@ def test_one_far_key_singled_out_among_hundreds(tier, dtype, target, portion):
 def test_router_takes_the_largest_scores_and_renormalises(tier):
     dev = _dev(tier)
     from colossalai_b200.models.config import ExpertFFSpec, ModelConfig
-    from colossalai_b200.models.moe import ClampedExpertFF
+    from colossalai_b200.models.moe import RoutedExpertFF
 
     torch.manual_seed(0)
     cfg = ModelConfig(hidden_size=32, vocab_size=16, num_hidden_layers=1, num_attention_heads=1)
     for dtype in (torch.float32, torch.bfloat16):
-        ff = ClampedExpertFF(cfg, ExpertFFSpec(experts=6, top=3, ff=8, limit=1.0, shared_ff=0)).to(dev).to(dtype)
+        ff = RoutedExpertFF(cfg, ExpertFFSpec(experts=6, top=3, ff=8, limit=1.0, shared_ff=0)).to(dev).to(dtype)
         with torch.no_grad():
             ff.router.weight.copy_(_rand(6, 32, seed=40, scale=0.7))
         x = _rand(9, 32, seed=41).to(dtype)
