@@ -6,9 +6,11 @@ at equal width and number of layer runs, and its kernels beside their like kerne
 for the Pogorax family (pairs of attention and a recurrent mixer side by side, selective state spaces, pre-norm layers),
 `--family domorax` for the Domorax family (windowed latent attention with sinks, convolved attention with distance slopes,
 delta rule with a decay per head, grouped output norms, a depth-weighted stream, normalised-power and routed feed-forwards).
+`--family sodurax` runs the Sodurax family (windowed attention that keeps the first keys, tanh norms on both sides of every
+sublayer, sigmoid-routed squared-ReLU experts, layers that run twice) beside Domorax, the closest served family.
 
     python examples/inference/benchmark_hybrid.py [--sizes 2048x8,4096x4] [--batch 8] [--in_len 2048] [--out_len 64]
-                                                  [--family gopunex|palilix|pogorax|domorax]
+                                                  [--family gopunex|palilix|pogorax|domorax|sodurax]
 
 Also reachable as `python bench.py --workload hybrid-serve`.  One JSON line per (size, family) and one per kernel.
 Timing: CUDA events on the launching stream after warm-up; the kernel timings write a 256 MB buffer between runs (L2
@@ -121,6 +123,24 @@ def domorax_config(width: int, layers: int, vocab: int = 32000, kv_rank: int = 1
                        depth_average=True, fp32_logits=True, max_position_embeddings=1 << 20)
 
 
+def sodurax_config(width: int, layers: int, vocab: int = 32000) -> ModelConfig:
+    """`layers` layer runs; the second half of them runs on the tensors of the first half.  Heads of 128 channels, one key
+    head per four query heads, the first 64 channels rotated with positions divided by 4, a window of 1024 positions beside
+    which the first 4 stay visible, an output gate.  Sixteen squared-ReLU experts of 1 x width (top 4) in four groups of
+    which two are open."""
+    H = width // 128
+    att = MixerSpec(kind="attention", heads=H, kv_heads=max(H // 4, 1), dim=128, vdim=128, bias=True, scale=128 ** -0.5,
+                    rot_dims=64, rot_base=5e5, rot_scaling=[4.0], window=1024, keep_first=4, out_gate=True, wide_weights=True)
+    moe = ExpertFFSpec(experts=16, top=4, ff=width, act="relu2", score="sigmoid", correction=True, renormalize=False, groups=4,
+                       keep_groups=2)
+    own = (layers + 1) // 2
+    return ModelConfig(model_type="sodurax", vocab_size=vocab, hidden_size=width, intermediate_size=width,
+                       layer_specs=[LayerSpec(mixer=att, moe=moe) for _ in range(own)],
+                       layer_order=[i % own for i in range(layers)], norm_eps=1e-5, norm_type="tanh", norm_placement="both",
+                       hidden_act="relu2", glu=False, pos_type="none", fp32_residual=True, fp32_logits=True,
+                       tie_word_embeddings=True, max_position_embeddings=1 << 20)
+
+
 def llama_config(width: int, layers: int, vocab: int = 32000) -> ModelConfig:
     H = width // 128
     # 8/3 x width gated feed-forward = the parameter count of the hybrid's 4 x width plain one
@@ -145,6 +165,8 @@ def build(cfg: ModelConfig):
                 p.copy_(torch.tensor([0.6, 0.3, 0.1, 0.0]))
             elif n.endswith("depth_weight"):
                 p.fill_(1.0 / p.numel())
+            elif n.endswith("correction"):
+                p.normal_(0, 0.2)
     return model.eval()
 
 
@@ -657,6 +679,118 @@ def kernels_domorax(width: int, batch: int, in_len: int, kv_rank: int = 192, rot
     return rows
 
 
+def kernels_sodurax(width: int, batch: int, in_len: int) -> list:
+    """Every kernel of the Sodurax layers alone at one layer's sizes beside its like kernel of the closest families."""
+    from colossalai_b200 import ops
+    from colossalai_b200.moe.grouped_gemm import grouped_linear
+    from colossalai_b200.ops import mixers as M
+    from colossalai_b200.ops import moe as MO
+
+    hbm, tflops, src = peaks()
+    dev, dt = "cuda", torch.bfloat16
+    H, d, bs = width // 128, 128, 64
+    G = max(H // 4, 1)
+    flush = torch.zeros(64 << 20, dtype=torch.float32, device=dev)
+    rows = []
+
+    def rec(name, phase, ms, bytes_, flops, like=""):
+        ideal = max(bytes_ / hbm, flops / tflops) * 1e3
+        rows.append({"kernel": name, "phase": phase + ("(graph replay)" if phase == "decode" else ""), "width": width,
+                     "ms": ms, "roofline_ms": ideal, "frac_of_" + src + "_roofline": ideal / ms,
+                     "bound": "hbm" if bytes_ / hbm > flops / tflops else "tensor", "like": like})
+
+    for phase, q_len, ctx in (("prefill", in_len, 0), ("decode", 1, in_len)):
+        replay = phase == "decode"             # decode kernels are timed as graph replays (no host share)
+        T = batch * q_len
+        L = ctx + q_len
+        meta = M.RaggedMeta.build([q_len] * batch, [ctx] * batch, list(range(batch)), dev)
+        x = lambda c: torch.randn(T, c, device=dev, dtype=dt)
+        t = lambda fn: _time(fn, flush, graph=replay)
+        # tanh norms around the stream's update  |  like: output norm + scaled add of Gopunex / Domorax
+        xs, y1, yf = torch.randn(T, width, device=dev), x(width), torch.randn(T, width, device=dev)
+        w, z = torch.ones(width, device=dev, dtype=dt), torch.zeros(width, device=dev, dtype=dt)
+        nrm = (torch.tensor(0.5, device=dev, dtype=dt), w, z)
+        rec("stream_tanh_norm(out + in)", phase, t(lambda: M.stream_tanh_norm(xs, y1, nrm, nrm)), T * width * (4 + 4 + 2 + 2), 0,
+            like="rmsnorm_residual")
+        rec("stream_tanh_norm(out + in, fp32 sum in)", phase, t(lambda: M.stream_tanh_norm(xs, yf, nrm, nrm)),
+            T * width * (4 + 4 + 4 + 2), 0, like="rmsnorm_residual(fp32 sum in)")
+        rec("gopunex:rmsnorm_residual", phase, t(lambda: M.rms_norm_residual(xs, y1, w, 1e-5, 0.7, 1.0)),
+            T * width * (4 + 4 + 2 + 2), 0)
+        rec("domorax:rmsnorm_residual(fp32 sum in)", phase, t(lambda: M.rms_norm_residual(xs, yf, w, 1e-5, 0.5, groups=4)),
+            T * width * (4 + 4 + 4 + 2), 0)
+        # rotation + page write in one pass  |  like: Llama's rotation, Gopunex page write
+        per = (L + bs - 1) // bs
+        kc, vc = (torch.randn(batch * per, bs, G, d, device=dev, dtype=dt) for _ in range(2))
+        tables = torch.arange(batch * per, dtype=torch.int32, device=dev).view(batch, per)
+        table = M.rotary_table(L + 1, 64, 5e5, dev, [4.0])
+        full = M.rotary_table(L + 1, d, 5e5, dev, [4.0])
+        qkv = x((2 * H + 2 * G) * d)
+        rec("rotary_kv_write(64 of 128)", phase,
+            t(lambda: M.rotary_kv_write(qkv, H, G, d, d, 64, table, kc, vc, tables, meta)),
+            T * (2 * H * 64 + 4 * G * d) * 2, 0, like="rope_qkv")
+        rec("rotary_kv_write(128 of 128)", phase,
+            t(lambda: M.rotary_kv_write(qkv, H, G, d, d, d, full, kc, vc, tables, meta)), T * (2 * H * d + 4 * G * d) * 2, 0,
+            like="rope_qkv")
+        cos, sin = ops.build_rope_cache(L + 1, d, 5e5, device=dev)
+        pos, ql = meta.token_pos.long(), x((H + 2 * G) * d)
+        rec("llama:rope_qkv", phase, t(lambda: ops.rope_qkv(ql, pos, cos, sin, H, G, d)), 2 * T * (H + G) * d * 2, 0)
+        kk, vv = ql[:, H * d:(H + G) * d], ql[:, (H + G) * d:]
+        rec("gopunex:paged_kv_write_mix", phase, t(lambda: M.paged_kv_write_mix(kk, vv, kc, vc, tables, meta)),
+            2 * T * 2 * G * d * 2, 0)
+        # attention: window 1024 + 4 kept keys, two-term weights  |  like: the same without window, Domorax slopes, Gopunex
+        win, keep = 1024, 4
+        seen = sum(min(p_ + 1, win + keep) for p_ in range(ctx, L)) * batch
+        qa = x(H * d)
+        io = 2 * T * H * d * 2
+        rec("paged_attention(window 1024, 4 kept, two-term weights)", phase,
+            t(lambda: M.paged_bias_attention(qa, kc, vc, tables, meta, d ** -0.5, window=win, keep_first=keep, wide_weights=True)),
+            2 * batch * min(L, win + keep + q_len) * G * d * 2 + io, 4.0 * H * d * seen,
+            like="paged_attention(distance slopes, two-term weights)")
+        every = batch * (q_len * ctx + q_len * (q_len + 1) / 2)
+        slopes = M.distance_slopes(H).to(dev)
+        rec("domorax:paged_attention(distance slopes, two-term weights)", phase,
+            t(lambda: M.paged_bias_attention(qa, kc, vc, tables, meta, d ** -0.5, slopes=slopes, wide_weights=True)),
+            2 * batch * L * G * d * 2 + io, 4.0 * H * d * every)
+        # (a latent row of 192 + 64 columns, window 1024, sinks)
+        lc = torch.randn(batch * per, bs, 1, 256, device=dev, dtype=dt)
+        qa2, sinks = x(H * 256), torch.randn(H, device=dev)
+        rec("domorax:latent_attention(window 1024, sinks, two-term weights)", phase,
+            t(lambda: M.paged_bias_attention(qa2, lc, lc, tables, meta, d ** -0.5, vdim=192, window=win, sink=True,
+                                             sink_values=sinks, wide_weights=True)),
+            batch * min(L, win + q_len) * 256 * 2 + T * H * 448 * 2,
+            2.0 * H * 448 * sum(min(p_ + 1, win) for p_ in range(ctx, L)) * batch)
+        gate = qkv[:, (H + 2 * G) * d:]
+        rec("sigmoid_gate_mul", phase, t(lambda: M.sigmoid_gate_mul(qa, gate)), 3 * T * H * d * 2, 0, like="(pogorax: same kernel)")
+        # router, squared ReLU, expert GEMMs, gather
+        E, top = 16, 4
+        logits, corr = torch.randn(T, E, device=dev), torch.randn(E, device=dev) * 0.2
+        rec("router_sigmoid(16, 4 groups, top 4)", phase, t(lambda: MO.router_sigmoid_topk(logits, top, corr, 4, 2)),
+            T * (E * 4 + top * 12), 0, like="router_topk")
+        rec("palilix:router_topk(16, top 4)", phase, t(lambda: MO.router_topk(logits, top)), T * (E * 4 + top * 12), 0)
+        u = torch.randn(T * top, width, device=dev, dtype=dt)
+        rec("bias_act(relu2)", phase, t(lambda: ops.bias_act(u, None, "relu2")), 2 * T * top * width * 2, 0, like="glu_fwd(silu)")
+        gu = torch.randn(T * top, 2 * width, device=dev, dtype=dt)
+        rec("domorax:glu_fwd(silu)", phase, t(lambda: ops.glu(gu, "silu")), 3 * T * top * width * 2, 0)
+        with torch.no_grad():
+            we = torch.randn(E, width, width, device=dev, dtype=dt) * 0.02
+            cnt = torch.full((E,), T * top // E, dtype=torch.int64, device=dev)
+            rec("grouped_gemm(expert up / down)", phase, t(lambda: grouped_linear(u, we, cnt)),
+                2 * T * top * width * 2 + E * width * width * 2, 2.0 * T * top * width * width, like="grouped_gemm(gate | up)")
+            wg = torch.randn(8, 2 * width, width, device=dev, dtype=dt) * 0.02
+            cg = torch.full((8,), T * 2 // 8, dtype=torch.int64, device=dev)
+            u2 = u[: 2 * T]
+            rec("domorax:grouped_gemm(gate | up)", phase, t(lambda: grouped_linear(u2, wg, cg)),
+                T * 2 * 3 * width * 2 + 8 * 2 * width * width * 2, 4.0 * T * 2 * width * width)
+        row_of, wts = torch.randperm(top * T, device=dev).view(T, top), torch.rand(T, top, device=dev)
+        rec("moe_gather_combine(top 4)", phase, t(lambda: MO.gather_combine(u, row_of, wts)), T * width * (top * 2 + 4), 0,
+            like="moe_gather_combine(+ gated shared expert)")
+        sh, sg = x(width), torch.randn(T, device=dev)
+        r2, w2 = torch.randperm(2 * T, device=dev).view(T, 2), torch.rand(T, 2, device=dev)
+        rec("domorax:moe_gather_combine(+ gated shared expert)", phase,
+            t(lambda: MO.gather_combine(u2, r2, w2, extra=sh, extra_gate=sg)), T * width * (3 * 2 + 4), 0)
+    return rows
+
+
 def main(argv=None):
     ap = argparse.ArgumentParser()
     ap.add_argument("--sizes", default="2048x8,4096x4", help="width x layers, comma separated")
@@ -664,9 +798,9 @@ def main(argv=None):
     ap.add_argument("--in_len", type=int, default=2048)
     ap.add_argument("--out_len", type=int, default=32)
     ap.add_argument("--cuda_graph", action="store_true", help="also run both families with CUDA-graph decode steps")
-    ap.add_argument("--family", default="gopunex", choices=["gopunex", "palilix", "pogorax", "domorax"],
+    ap.add_argument("--family", default="gopunex", choices=["gopunex", "palilix", "pogorax", "domorax", "sodurax"],
                     help="gopunex: the hybrid decoder beside Llama (default).  palilix / pogorax / domorax: that family "
-                         "beside Gopunex, the closest served family")
+                         "beside Gopunex, the closest served family; sodurax: beside Domorax")
     ap.add_argument("--no-kernels", action="store_true")
     ap.add_argument("--no-serve", action="store_true")
     args = ap.parse_args(argv)
@@ -678,12 +812,13 @@ def main(argv=None):
                 pair = {"gopunex": lambda: (hybrid_config(width, layers), llama_config(width, layers)),
                         "palilix": lambda: (palilix_config(width, layers), hybrid_config(width, layers)),
                         "pogorax": lambda: (pogorax_config(width, layers), hybrid_config(width, layers)),
-                        "domorax": lambda: (domorax_config(width, layers), hybrid_config(width, layers))}[args.family]()
+                        "domorax": lambda: (domorax_config(width, layers), hybrid_config(width, layers)),
+                        "sodurax": lambda: (sodurax_config(width, layers), domorax_config(width, layers))}[args.family]()
                 for cfg in pair:
                     print(json.dumps(serve(cfg, args.batch, args.in_len, args.out_len, graph)), flush=True)
         if not args.no_kernels:
             kfn = {"gopunex": kernels, "palilix": kernels_palilix, "pogorax": kernels_pogorax,
-                   "domorax": kernels_domorax}[args.family]
+                   "domorax": kernels_domorax, "sodurax": kernels_sodurax}[args.family]
             for row in kfn(width, args.batch, args.in_len):
                 print(json.dumps(row), flush=True)
 
