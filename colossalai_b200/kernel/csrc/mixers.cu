@@ -1814,8 +1814,8 @@ __global__ void __launch_bounds__(128) attention_merge_kernel(const float* __res
   const int blk_lo = att_first_key(tpos - nth + row0 / R, mask_block, window) / MMA_BN * MMA_BN;
   const int nkept = att_kept_tiles(keep_first, blk_lo);
   const int nsp = min((nkept + (tpos - blk_lo) / MMA_BN) / ct + 1, max_splits);
-  // first chunk with a visible key
-  const int sp0 = nkept > 0 ? 0 : (att_first_key(tpos, mask_block, window) - blk_lo) / MMA_BN / ct;
+  // first chunk with a visible key (kept first keys sit at the start of the list, also where the range itself starts at 0)
+  const int sp0 = keep_first > 0 ? 0 : (att_first_key(tpos, mask_block, window) - blk_lo) / MMA_BN / ct;
   const float* ml = part_ml + unit * max_splits * 2;
   const float sk = sink_vals != nullptr ? sink_vals[unit % heads] * 1.4426950408889634f : 0.f;
   float mm = sink ? sk : -INFINITY;
@@ -2141,8 +2141,9 @@ __global__ void __launch_bounds__(256) sigmoid_gate_mul_kernel(T* __restrict__ o
 // ------------------------------------------------------------------------------------------------ tanh norms of the stream
 // n(z) = tanh(alpha z) w + b with a scalar alpha and vectors w, b (fp32 or T): no statistics over the row, so the norm of a
 // sublayer's output, its addition to the fp32 stream and the norm in front of the next sublayer are one elementwise pass.
-// A thread keeps the parameters of its VEC columns in registers and walks over the rows, TANH_ROWS of them in flight.
-constexpr int TANH_ROWS = 2;
+// A thread keeps the parameters of its VEC columns in registers and walks over the rows, ROWS of them in flight (a 16-bit y
+// takes eight columns of one row, an fp32 y four columns of two rows: measured best of seven shapes; more values per thread
+// cost the occupancy that hides tanh's latency).
 
 struct TanhNorm {
   const void *alpha, *w, *b;    // w == nullptr: absent
@@ -2162,7 +2163,7 @@ template <typename T, int VEC> struct TanhParams {
   CB_DEVICE float operator()(float z, int e) const { return fmaf(tanhf(a * z), w[e], b[e]); }
 };
 
-template <typename T, int VEC>
+template <typename T, int VEC, int ROWS>
 __global__ void __launch_bounds__(128) stream_tanh_norm_kernel(float* __restrict__ x, const void* __restrict__ y,
                                                                int64_t ldy, int y_f32, TanhNorm no, TanhNorm ni,
                                                                void* __restrict__ h, int h_f32, int64_t tokens, int W) {
@@ -2171,16 +2172,16 @@ __global__ void __launch_bounds__(128) stream_tanh_norm_kernel(float* __restrict
   TanhParams<T, VEC> po, pi;
   po.load(no, c);
   pi.load(ni, c);
-  for (int64_t t0 = (int64_t)blockIdx.y * TANH_ROWS; t0 < tokens; t0 += (int64_t)gridDim.y * TANH_ROWS) {
-    float xv[TANH_ROWS][VEC], yv[TANH_ROWS][VEC];
+  for (int64_t t0 = (int64_t)blockIdx.y * ROWS; t0 < tokens; t0 += (int64_t)gridDim.y * ROWS) {
+    float xv[ROWS][VEC], yv[ROWS][VEC];
 #pragma unroll
-    for (int r = 0; r < TANH_ROWS; ++r)
+    for (int r = 0; r < ROWS; ++r)
       if (t0 + r < tokens) {
         load_vec<T, VEC>(x, true, (t0 + r) * W + c, xv[r]);
         if (y != nullptr) load_vec<T, VEC>(y, y_f32 != 0, (t0 + r) * ldy + c, yv[r]);
       }
 #pragma unroll
-    for (int r = 0; r < TANH_ROWS; ++r)
+    for (int r = 0; r < ROWS; ++r)
       if (t0 + r < tokens) {
         if (y != nullptr) {
 #pragma unroll
@@ -2792,15 +2793,17 @@ int cb_stream_tanh_norm(float* x, const void* y, int64_t ldy, int y_f32, const v
   const TanhNorm no{oa, ow, ob, p_f32}, ni{ia, iw, ib, p_f32};
   auto al = [](const void* p) { return ((uintptr_t)p & 15) == 0; };
   const bool vec = W % 4 == 0 && ldy % 4 == 0 && al(x) && al(y) && al(ow) && al(ob) && al(iw) && al(ib) && al(h);
-  const int cols = vec ? 128 * 4 : 128;
+  const bool wide = vec && dtype != CB_F32 && !p_f32 && !y_f32 && !h_f32 && W % 8 == 0 && ldy % 8 == 0 && ((uintptr_t)x & 31) == 0;
+  const int cols = 128 * (wide ? 8 : vec ? 4 : 1), rows = wide ? 1 : 2;
   const int gx = (W + cols - 1) / cols;
-  int64_t gy = (tokens + TANH_ROWS - 1) / TANH_ROWS;
+  int64_t gy = (tokens + rows - 1) / rows;
   const int64_t cap = (148 * 16 + gx - 1) / gx;
   if (gy > cap) gy = cap;
   dim3 grid(gx, (unsigned)gy);
   CB_DISPATCH_FLOAT(dtype, T, {
-    if (vec) stream_tanh_norm_kernel<T, 4><<<grid, 128, 0, st>>>(x, y, ldy, y_f32, no, ni, h, h_f32, tokens, W);
-    else stream_tanh_norm_kernel<T, 1><<<grid, 128, 0, st>>>(x, y, ldy, y_f32, no, ni, h, h_f32, tokens, W);
+    if (wide) stream_tanh_norm_kernel<T, 8, 1><<<grid, 128, 0, st>>>(x, y, ldy, y_f32, no, ni, h, h_f32, tokens, W);
+    else if (vec) stream_tanh_norm_kernel<T, 4, 2><<<grid, 128, 0, st>>>(x, y, ldy, y_f32, no, ni, h, h_f32, tokens, W);
+    else stream_tanh_norm_kernel<T, 1, 2><<<grid, 128, 0, st>>>(x, y, ldy, y_f32, no, ni, h, h_f32, tokens, W);
   });
   return CB_LAUNCH_CHECK();
 }

@@ -334,21 +334,28 @@ def test_spec_refuses_choices_that_cannot_be_made():
 
 # ------------------------------------------------------------------------------------------------ the kernels against each other
 @pytest.mark.gpu
+@pytest.mark.parametrize("H,G", [(4, 2), (2, 2), (3, 1)])
 @pytest.mark.parametrize("window,keep,L,dim,vdim", [(0, 0, 300, 32, 32), (24, 4, 300, 64, 64), (200, 70, 460, 40, 24),
                                                     (130, 1, 700, 160, 128), (72, 300, 900, 64, 64), (1, 64, 400, 128, 128)])
-def test_tensor_core_attention_against_the_exact_kernel(window, keep, L, dim, vdim):
+def test_tensor_core_attention_against_the_exact_kernel(window, keep, L, dim, vdim, H, G):
     """16-bit pages through the tensor-core kernel - kept keys in tiles of their own, inside the window's first tile and
-    over several tiles, long portions whose few row tiles split their tile lists over CTAs, decoded tokens, two unequal
-    sequences - row by row against the exact kernel on the same pages."""
+    over several tiles, long portions whose few row tiles split their tile lists over CTAs (also tiles of rows so far apart
+    that the first ones still start at key 0 while the last ones' windows start chunks later), decoded tokens, two unequal
+    sequences - row by row against the exact kernel on the same pages.  The kept keys score high: missing ones show."""
     dev = _dev("gpu")
-    H, G, bs = 4, 2, 16
+    bs = 16
     nb = L // bs + 1
     kc = _rand(2 * nb, bs, G, dim, seed=1).to(dev).to(torch.bfloat16)
     vc = _rand(2 * nb, bs, G, vdim, seed=2).to(dev).to(torch.bfloat16)
     tables = torch.arange(2 * nb, dtype=torch.int32, device=dev).view(2, -1)
-    for q_lens, ctx in [([L], [0]), ([1], [L - 1]), ([1, 1], [L - 1, 7]), ([5, 130], [L - 5, L - 130]), ([17], [L - 17])]:
+    toward = _rand(1, H // G, 1, dim, seed=4)                        # the direction all queries and the first keys share
+    for i in range(2):
+        for j in range(min(max(keep, 1), 3)):
+            kc[i * nb, j] += toward[0, 0].to(dev).to(torch.bfloat16) * 0.5
+    for q_lens, ctx in [([L], [0]), ([1], [L - 1]), ([1, 1], [L - 1, 7]), ([5, 130], [L - 5, L - 130]), ([17], [L - 17]),
+                        ([200], [0]), ([130, 1], [20, 50])]:
         meta = M.RaggedMeta.build(q_lens, ctx, list(range(len(q_lens))), dev)
-        q = _rand(sum(q_lens), H * dim, seed=3).to(dev).to(torch.bfloat16)
+        q = (_rand(sum(q_lens), H * dim, seed=3) + toward[0, 0].repeat(1, H) * 0.5).to(dev).to(torch.bfloat16)
         kw = dict(window=window, keep_first=keep)
         exact = M.paged_bias_attention(q, kc, vc, tables, meta, 0.2, tensor_cores=False, **kw).float()
         got = M.paged_bias_attention(q, kc, vc, tables, meta, 0.2, tensor_cores=True, wide_weights=True, **kw).float()
