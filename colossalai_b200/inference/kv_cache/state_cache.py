@@ -1,10 +1,10 @@
 """Fixed-size recurrent state per live sequence, beside the paged K / V of attention layers.
 
 A recurrent mixer (linear attention, retention, delta rule, selective state space, gated matrix memory, gated linear
-recurrence; also attention whose q / k pass a short convolution, which carries the convolution's window only) keeps, per sequence, fp32 memories ("S" and, for the gated matrix memory, the normaliser "n" and the running
+recurrence or attention; also attention behind a short convolution, which carries the convolution's window only) keeps, per sequence, fp32 memories ("S" and, for the gated matrix memory, the normaliser "n" and the running
 maximum "m") and - where it has short convolutions - the last few inputs of every convolved channel ("conv", in the
 compute dtype).  A layer whose mixer is a pair of mixers holds the pages of its paged part and the state of its recurrent
-part.  The pool holds `max_batch_size` slots per such
+parts (tensor names tagged by part where several keep state).  The pool holds `max_batch_size` slots per such
 layer; a sequence takes a slot when it is admitted and gives it back when it ends.  Slots are not cleared: the kernels
 take the state of a sequence that has consumed no token yet as zero.
 
@@ -58,11 +58,14 @@ def layer_state_shapes(model_config, layer: int, slots: int) -> Optional[Dict[st
     """Shapes of a recurrent layer's state tensors ("S", "n", "m": fp32 memories; "conv": carried convolution inputs in
     the compute dtype)."""
     sp = _spec(model_config, layer)
-    sp = None if sp is None else sp.recurrent_part
-    if sp is None:
-        return None
-    if sp.kind == "attention":            # attention behind a convolution on q | k: only the convolution's window
-        return {"conv": (slots, max(sp.conv - 1, 0), (sp.heads + sp.kv_heads) * sp.dim)}
+    parts = [] if sp is None else sp.recurrent_parts
+    return {n + tag: shape for tag, part in parts for n, shape in _mixer_state_shapes(part, slots).items()} or None
+
+
+def _mixer_state_shapes(sp, slots: int) -> Dict[str, Tuple[int, ...]]:
+    if sp.kind == "attention":            # attention behind a convolution on q | k (| v): only the convolution's window
+        return {"conv": (slots, max(sp.conv - 1, 0),
+                         (sp.heads + sp.kv_heads) * sp.dim + (sp.kv_heads * sp.vdim if sp.conv_values else 0))}
     if sp.kind == "rglru":
         return {"S": (slots, sp.lru_width), "conv": (slots, max(sp.conv - 1, 0), sp.lru_width)}
     if sp.kind == "ssd":

@@ -102,16 +102,18 @@ class PagedKVRuntime:
 
     def attend_latent(self, layer_idx: int, q: torch.Tensor, scale: float, kv_rank: int, window: int = 0,
                       sink: bool = False, sink_values: Optional[torch.Tensor] = None,
-                      wide_weights: bool = False) -> torch.Tensor:
+                      wide_weights: bool = False, head_gate: Optional[torch.Tensor] = None) -> torch.Tensor:
         """Latent attention over the layer's pages (rows [latent | rotated key part], written by the caller through
         `latent_cache`): q [T, H x (kv_rank + rot)] against the whole row, values = the row's first `kv_rank` columns;
-        optionally inside a sliding `window` and with a sink (`sink_values`: its score per head) in the denominator.
+        optionally inside a sliding `window`, with a sink (`sink_values`: its score per head) in the denominator and a
+        sigmoid gate per head (`head_gate`).
         Returns [T, H x kv_rank]."""
         from ...ops import mixers as mops
 
         kc = self.k_caches[self.cache_index(layer_idx)]
         return mops.paged_bias_attention(q, kc, kc, self.block_tables, self.ragged, scale, vdim=kv_rank, window=window,
-                                         sink=sink, sink_values=sink_values, wide_weights=wide_weights)
+                                         sink=sink, sink_values=sink_values, wide_weights=wide_weights,
+                                         head_gate=head_gate)
 
     def pages(self, layer_idx: int):
         """(key pages, value pages) of the layer's current run, for a mixer whose kernels write the step's rows themselves."""
@@ -124,11 +126,13 @@ class PagedKVRuntime:
                       bias_table=None, bucket_starts=None, sink: bool = False, v_other=None,
                       lam: float = 0.0, lut=None, mask_block: int = 0, wide_weights: bool = False,
                       sink_values: Optional[torch.Tensor] = None, slopes: Optional[torch.Tensor] = None,
-                      window: int = 0, keep_first: int = 0) -> torch.Tensor:
+                      window: int = 0, keep_first: int = 0, softcap: float = 0.0,
+                      head_gate: Optional[torch.Tensor] = None) -> torch.Tensor:
         """Write the step's K / V rows (values optionally blended with `v_other`) into the layer's pages, then attend
         every step token over positions 0..pos of its sequence (with `mask_block`: over the positions of its own block
         of that many positions only; with `window`: over the last `window` positions, with `keep_first` also over the
-        first that many of the sequence; `slopes`: a linear distance penalty per head; `sink_values`: the sink's score per head).  q [T, H x dim], k [T, G x dim], v [T, G x vdim];
+        first that many of the sequence; `slopes`: a linear distance penalty per head; `softcap`: scores through cap x tanh(. / cap); `sink_values`: the sink's
+        score per head; `head_gate`: one sigmoid gate per head on its output).  q [T, H x dim], k [T, G x dim], v [T, G x vdim];
         k = None: the caller has written the step's rows itself (`pages`)."""
         from ...ops import mixers as mops
 
@@ -138,7 +142,7 @@ class PagedKVRuntime:
         return mops.paged_bias_attention(q, kc, vc, self.block_tables, self.ragged, scale, bias_table=bias_table,
                                          bucket_starts=bucket_starts, sink=sink, lut=lut, mask_block=mask_block,
                                          wide_weights=wide_weights, sink_values=sink_values, slopes=slopes, window=window,
-                                         keep_first=keep_first)
+                                         keep_first=keep_first, softcap=softcap, head_gate=head_gate)
 
     @classmethod
     def scratch(cls, cfg, batch: int, seqlen: int, device, dtype, block_size: int = 16) -> "PagedKVRuntime":

@@ -17,7 +17,8 @@
 //                           per head; or the gated delta rule M <- diag(r) M; e = w (v - M^T k); M <- M + outer(k, e)
 //                           with a decay per key channel; or M <- g_t M + w_t outer(k, v) with a decay g_t and a write
 //                           strength w_t per token and head (selective state space: from the step size; matrix memory
-//                           with exponential gates: from a running maximum, with a normaliser vector beside M); the
+//                           with exponential gates: from a running maximum, with a normaliser vector beside M); or
+//                           M <- diag(r_t) M + outer(k, v) with a decay per key channel (gated linear attention); the
 //                           read-out y = M^T q follows the write
 //   cb_lru_scan             per channel S <- a_t S + sqrt(1 - a_t^2) i_t u_t with gates from fp32 pre-activations
 //   cb_gated_group_rmsnorm  out = o / rms_group(o) * w * sigmoid(gate) (or silu(gate); w optional; gate before or
@@ -27,7 +28,8 @@
 //   cb_norm_mean            mean of up to four RMS-normed [T, W] tensors, fp32 out
 //   cb_sigmoid_gate_mul     o *= sigmoid(gate)
 //   cb_stream_add_norm      x(fp32) += sum of up to four [T, W] addends + a [W] row;  h = cast(rms / layer norm of x)
-//   cb_rotary_half          rotate-half rotary positions from an fp32 [positions, dims] cos|sin table, strided in / out
+//   cb_rotary_half          rotary positions (half or interleaved pairs) from an fp32 [positions, dims] cos|sin table,
+//                           strided in / out
 //   cb_latent_kv_write      latent attention's cache row: [rms_norm(latent) * w | rotated shared key part]
 //   cb_clamped_glu          g = min(gate, L); u = clamp(up, -L, L); out = g * sigmoid(alpha g) * (u + 1)
 //   cb_rmsnorm_residual     x(fp32) += mult * y / rms(y) * (offset + w);  h = cast(x)
@@ -35,11 +37,13 @@
 //   cb_paged_kv_write_mix   K / V rows (different widths allowed) into the paged cache, V optionally blended with another
 //                           layer's values first
 //   cb_paged_bias_attention causal attention of every step token over its sequence's paged cache with
-//                           score = scale * q.k + table[bucket(distance)][head] - slope[head] * distance, an optional
-//                           sink (score 0 or learned per head) in the denominator, a block mask or a sliding window
+//                           score = scale * q.k + table[bucket(distance)][head] - slope[head] * distance, optionally
+//                           soft-capped scale * q.k, an optional sink (score 0 or learned per head) in the denominator,
+//                           a block mask or a sliding window, a sigmoid gate per head on the output
 //   cb_stream_tanh_norm     x(fp32) += y or n_o(y);  h = cast(n_i(x)), n(z) = tanh(alpha z) w + b element by element
 //   cb_router_sigmoid       sigmoid router scores, choice by score + correction inside the best groups of experts
 //   cb_rotary_kv_write      q heads rotated in place, rotated k heads and v heads into their pages, one pass over q | k | v
+//   cb_conv_rotary_kv_write the same behind a short convolution on q | k | v, with a unit norm of the q / k heads
 //   cb_depth_mix            weighted sum over the history of the fp32 stream (+ compute-dtype copy)
 //   cb_poly_norm            a N(z) + b N(z^2) + c N(z^3) + e with N = division by the row's root mean square
 //   cb_head_rmsnorm         RMS norm per head with a weight over the head's channels (query heads | key heads); optionally
@@ -206,7 +210,7 @@ __global__ void __launch_bounds__(128) short_conv_state_kernel(const T* __restri
 }
 
 // ------------------------------------------------------------------------------------------------ recurrent state scan
-enum ScanMode : int { SCAN_DECAY = 0, SCAN_DELTA = 1, SCAN_GATED = 2 };
+enum ScanMode : int { SCAN_DECAY = 0, SCAN_DELTA = 1, SCAN_GATED = 2, SCAN_ROWS = 3 };
 enum GateKind : int { GATE_STEP = 1, GATE_EXP = 2, GATE_HEAD = 3 };
 constexpr int SCAN_TOK_TILE = 8;
 
@@ -240,6 +244,9 @@ struct ScanParams {
   float gate_cap;
   float* state_n;
   float* state_m;
+  // rows mode (gated linear attention): araw [T, lda] fp32 holds heads x dim pre-activations, dt_bias [heads x dim] their
+  // biases: row decay = sigmoid(araw + dt_bias)^(1 / tau)
+  float inv_tau;
 };
 
 // Two kernels.  `scan_prepare_kernel` is elementwise and fully parallel: activations, unit norms, decays and write
@@ -321,6 +328,13 @@ __global__ void __launch_bounds__(128) scan_prepare_kernel(ScanParams p, ScanWor
     }
     for (int h = threadIdx.x; h < p.heads; h += blockDim.x)
       w.beta[t * p.heads + h] = sigmoid_f(to_f32<T>(((const T*)p.braw)[t * p.ldb + h]));
+  }
+  if (MODE == SCAN_ROWS) {
+    const float* ar = (const float*)p.araw + t * p.lda;
+    for (int h = warp; h < p.heads; h += nwarps)
+      for (int i = lane; i < DK; i += 32)
+        w.g[(t * p.heads + h) * DK + i] =
+            i < dim ? expf(logsigmoid_f(ar[h * dim + i] + p.dt_bias[h * dim + i]) * p.inv_tau) : 1.f;
   }
   if (MODE == SCAN_GATED) {
     const T* ar = (const T*)p.araw + t * p.lda;
@@ -422,7 +436,8 @@ __global__ void __launch_bounds__(128, DK > 128 ? 2 : 4) state_scan_kernel(ScanP
   constexpr int RP = DK / SCAN_PARTS;  // rows per lane
   constexpr int RPP = RP + 4;          // a lane's rows start 4 floats further: the four 16-byte reads of a warp hit
   constexpr int DKP = SCAN_PARTS * RPP;  // different banks
-  constexpr int NROW = MODE == SCAN_DELTA ? 3 : 2;
+  constexpr bool ROWS = MODE == SCAN_DELTA || MODE == SCAN_ROWS;        // decay rows beside q and k
+  constexpr int NROW = ROWS ? 3 : 2;
   constexpr int STAGE = SCAN_TOK_TILE * (NROW * DKP + SCAN_COLS + 4);     // floats per stage
   extern __shared__ __align__(16) float scan_smem[];
   const int vblocks = w.VP / SCAN_COLS;
@@ -455,7 +470,7 @@ __global__ void __launch_bounds__(128, DK > 128 ? 2 : 4) state_scan_kernel(ScanP
       const int64_t t = tb + tt;
       cp_async16f(base + dst, w.q + (t * p.qk_heads + hk) * DK + c);
       cp_async16f(base + SCAN_TOK_TILE * DKP + dst, w.k + (t * p.qk_heads + hk) * DK + c);
-      if (MODE == SCAN_DELTA) cp_async16f(base + 2 * SCAN_TOK_TILE * DKP + dst, w.g + (t * p.heads + h) * DK + c);
+      if (ROWS) cp_async16f(base + 2 * SCAN_TOK_TILE * DKP + dst, w.g + (t * p.heads + h) * DK + c);
     }
     float* sv = base + NROW * SCAN_TOK_TILE * DKP;
     for (int idx = threadIdx.x; idx < nt * (SCAN_COLS / 4); idx += blockDim.x) {
@@ -529,6 +544,18 @@ __global__ void __launch_bounds__(128, DK > 128 ? 2 : 4) state_scan_kernel(ScanP
           o0 = fmaf(S[i], q4.x, o0); o1 = fmaf(S[i + 1], q4.y, o1);
           o0 = fmaf(S[i + 2], q4.z, o0); o1 = fmaf(S[i + 3], q4.w, o1);
         }
+      } else if (MODE == SCAN_ROWS) {
+        const float* gq = sg + tt * DKP + r0p;
+#pragma unroll
+        for (int i = 0; i < RP; i += 4) {
+          const float4 g4 = *reinterpret_cast<const float4*>(gq + i);
+          const float4 k4 = *reinterpret_cast<const float4*>(kq + i);
+          const float4 q4 = *reinterpret_cast<const float4*>(qq + i);
+          S[i] = fmaf(g4.x, S[i], k4.x * vv); S[i + 1] = fmaf(g4.y, S[i + 1], k4.y * vv);
+          S[i + 2] = fmaf(g4.z, S[i + 2], k4.z * vv); S[i + 3] = fmaf(g4.w, S[i + 3], k4.w * vv);
+          o0 = fmaf(S[i], q4.x, o0); o1 = fmaf(S[i + 1], q4.y, o1);
+          o0 = fmaf(S[i + 2], q4.z, o0); o1 = fmaf(S[i + 3], q4.w, o1);
+        }
       } else {
 #pragma unroll
         for (int i = 0; i < RP; i += 4) {
@@ -557,7 +584,7 @@ __global__ void __launch_bounds__(128, DK > 128 ? 2 : 4) state_scan_kernel(ScanP
 
 template <int DK, int MODE> int launch_scan_dk(const ScanParams& p, const ScanWork& w, int nseq, cudaStream_t st) {
   constexpr int DKP = SCAN_PARTS * (DK / SCAN_PARTS + 4);
-  constexpr int NROW = MODE == SCAN_DELTA ? 3 : 2;
+  constexpr int NROW = MODE == SCAN_DELTA || MODE == SCAN_ROWS ? 3 : 2;
   const size_t smem = (size_t)2 * SCAN_TOK_TILE * (NROW * DKP + SCAN_COLS + 4) * sizeof(float);
   auto kern = state_scan_kernel<DK, MODE>;
   static bool configured = false;
@@ -571,7 +598,7 @@ template <int DK, int MODE> int launch_scan_dk(const ScanParams& p, const ScanWo
   return CB_LAUNCH_CHECK();
 }
 
-// workspace floats for `tokens` tokens: q, k rows, decay rows and write strengths (delta rule), value rows
+// workspace floats for `tokens` tokens: q, k rows, decay rows (delta rule, rows mode), write strengths (delta rule), value rows
 static inline int scan_dk(int dim) { return dim <= 16 ? 16 : dim <= 32 ? 32 : dim <= 64 ? 64 : dim <= 128 ? 128 : 256; }
 static inline int scan_vp(int vdim) { return (vdim + SCAN_COLS - 1) / SCAN_COLS * SCAN_COLS; }
 
@@ -584,7 +611,7 @@ int launch_scan(const ScanParams& p, float* work, int64_t tokens, int nseq, cuda
   w.q = work;
   w.k = w.q + tokens * p.qk_heads * w.DK;
   w.g = w.k + tokens * p.qk_heads * w.DK;
-  w.beta = w.g + (MODE == SCAN_DELTA ? tokens * p.heads * w.DK : 0);
+  w.beta = w.g + (MODE == SCAN_DELTA || MODE == SCAN_ROWS ? tokens * p.heads * w.DK : 0);
   w.gw = w.beta;
   w.v = w.beta + (MODE == SCAN_DELTA ? (tokens * p.heads + 3) / 4 * 4 : (MODE == SCAN_GATED ? tokens * p.heads * 4 : 0));
   scan_prepare_kernel<MODE, T><<<(unsigned)tokens, 128, 0, st>>>(p, w);
@@ -1124,12 +1151,12 @@ template <typename T, int NORM> int launch_stream_add_norm(const StreamArgs& g, 
 // ------------------------------------------------------------------------------------------------ rotary positions
 // table [positions, dims] fp32: cos(p f_i) for i < dims / 2, then sin(p f_i).  A work item is VEC consecutive channels of
 // one (token, head): in the rotated part the item takes channels i.. of the first half TOGETHER with their partners
-// i + dims / 2.. (two loads, two stores of VEC values); behind the rotated part it copies.  VEC = 8 (16-byte accesses of
+// i + dims / 2.. (two loads, two stores of VEC values), with interleaved pairs (2i, 2i + 1) 2 VEC adjacent channels; behind the rotated part it copies.  VEC = 8 (16-byte accesses of
 // 16-bit data) when every offset, stride and width allows it, else 1.
 template <typename T, int VEC>
 __global__ void __launch_bounds__(256) rotary_half_kernel(const T* __restrict__ src, int64_t lds, T* __restrict__ dst,
                                                           int64_t ldd, int64_t tokens, int heads, int src_hs, int src_off,
-                                                          int dst_hs, int dst_off, int width, int dims,
+                                                          int dst_hs, int dst_off, int width, int dims, int interleaved,
                                                           const float* __restrict__ table,
                                                           const int* __restrict__ token_pos) {
   struct alignas(sizeof(T) * VEC) Pack { T v[VEC]; };
@@ -1145,6 +1172,21 @@ __global__ void __launch_bounds__(256) rotary_half_kernel(const T* __restrict__ 
     const int c = it * VEC;
     if (c < half) {
       const float* cs = table + (int64_t)token_pos[t] * dims;
+      if (interleaved) {                                     // pairs c .. c + VEC - 1 = channels 2c .. 2c + 2 VEC - 1
+        alignas(16) T in[2 * VEC], o[2 * VEC];
+        *reinterpret_cast<Pack*>(in) = *reinterpret_cast<const Pack*>(s + 2 * c);
+        *reinterpret_cast<Pack*>(in + VEC) = *reinterpret_cast<const Pack*>(s + 2 * c + VEC);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) {
+          const float co = cs[c + e], sn = cs[half + c + e];
+          const float uf = to_f32<T>(in[2 * e]), vf = to_f32<T>(in[2 * e + 1]);
+          o[2 * e] = from_f32<T>(uf * co - vf * sn);
+          o[2 * e + 1] = from_f32<T>(vf * co + uf * sn);
+        }
+        *reinterpret_cast<Pack*>(d + 2 * c) = *reinterpret_cast<const Pack*>(o);
+        *reinterpret_cast<Pack*>(d + 2 * c + VEC) = *reinterpret_cast<const Pack*>(o + VEC);
+        continue;
+      }
       const Pack u = *reinterpret_cast<const Pack*>(s + c);
       const Pack v = *reinterpret_cast<const Pack*>(s + c + half);
       Pack ou, ov;
@@ -1170,7 +1212,7 @@ __global__ void __launch_bounds__(256) rotary_half_kernel(const T* __restrict__ 
 // accesses; the launcher checks widths and alignment), else VEC = 1.
 template <typename T, typename TW, int VEC>
 __global__ void __launch_bounds__(256) latent_kv_write_kernel(const T* __restrict__ z, int64_t ldz, const TW* __restrict__ w,
-                                                              float eps, int rank, int rot,
+                                                              float eps, int rank, int rot, int interleaved,
                                                               const float* __restrict__ table, T* __restrict__ cache,
                                                               const int* __restrict__ block_tables,
                                                               const int* __restrict__ token_seq,
@@ -1218,10 +1260,11 @@ __global__ void __launch_bounds__(256) latent_kv_write_kernel(const T* __restric
   const int half = rot >> 1;
   const float* cs = table + (int64_t)pos * rot;
   for (int i = lane; i < half; i += 32) {
-    const float u = to_f32<T>(zr[rank + i]), v = to_f32<T>(zr[rank + half + i]);
+    const int iu = rank + (interleaved ? 2 * i : i), iv = interleaved ? iu + 1 : iu + half;
+    const float u = to_f32<T>(zr[iu]), v = to_f32<T>(zr[iv]);
     const float c = cs[i], sn = cs[half + i];
-    out[rank + i] = from_f32<T>(u * c - v * sn);
-    out[rank + half + i] = from_f32<T>(v * c + u * sn);
+    out[iu] = from_f32<T>(u * c - v * sn);
+    out[iv] = from_f32<T>(v * c + u * sn);
   }
 }
 
@@ -1277,7 +1320,9 @@ __global__ void __launch_bounds__(128) paged_kv_write_mix_kernel(const T* __rest
 // (lane = key for the scores, lane = value channel for the weighted sum), online softmax in fp32.  With `sink` the running
 // maximum starts at the sink's score (`sink_vals[head]`, 0 without the table) and the denominator at 1: a key of that
 // score without a value, not scaled.  `slopes[head]` takes slope * (pos - key) off every score; `window` > 0 keeps the
-// keys pos - window + 1 .. pos and, whatever their distance, the first `keep_first` keys of the sequence.
+// keys pos - window + 1 .. pos and, whatever their distance, the first `keep_first` keys of the sequence.  `softcap` > 0 passes
+// the scaled product through softcap * tanh(. / softcap) first; `gate` [tokens, ldg] multiplies head h's output by
+// sigmoid(gate[t][h]).
 constexpr int ATT_MAX_VREG = 16;  // value width up to 512
 
 // first key of the contiguous range that ends at position p: the start of p's own block (block mask), the first key of
@@ -1295,7 +1340,7 @@ __global__ void __launch_bounds__(128) paged_bias_attention_kernel(
     const float* __restrict__ bias_table, const int* __restrict__ bucket_start, int nbuckets, T* __restrict__ out,
     int64_t tokens, int heads, int kv_heads, int dim, int vdim, int ldv, int block_size, int max_blocks, float scale,
     int sink, int mask_block, const float* __restrict__ sink_vals, const float* __restrict__ slopes, int window,
-    int keep_first) {
+    int keep_first, float softcap, const T* __restrict__ gate, int64_t ldg) {
   extern __shared__ float smem[];
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
   float* qs = smem + warp * dim;
@@ -1337,6 +1382,7 @@ __global__ void __launch_bounds__(128) paged_bias_attention_kernel(
       }
       if (i < dim) d0 = fmaf(qs[i], to_f32<T>(kr[i]), d0);
       sc = d0 + d1;
+      if (softcap > 0.f) sc = softcap * tanhf(sc / softcap);
       if (nbuckets > 0) {
         const int n = pos - jk;
         int b = n;
@@ -1367,7 +1413,8 @@ __global__ void __launch_bounds__(128) paged_bias_attention_kernel(
       }
     }
   }
-  const float inv = 1.f / l;
+  float inv = 1.f / l;
+  if (gate != nullptr) inv *= sigmoid_f(to_f32<T>(gate[t * ldg + h]));
 #pragma unroll
   for (int r = 0; r < ATT_MAX_VREG; ++r) {
     const int c = lane + 32 * r;
@@ -1417,6 +1464,15 @@ CB_DEVICE float ex2f(float x) {
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
+CB_DEVICE float rcpf(float x) {                 // 1 / inf = 0
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+// head h's gate of token t (1 without gates)
+template <typename T> CB_DEVICE float head_gate(const T* gate, int64_t ldg, int64_t t, int h) {
+  return gate != nullptr ? sigmoid_f(to_f32<T>(gate[t * ldg + h])) : 1.f;
+}
 CB_DEVICE void cp_async16(void* smem_dst, const void* gmem_src, uint32_t src_bytes) {
   const uint32_t dst = (uint32_t)__cvta_generic_to_shared(smem_dst);
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(gmem_src), "r"(src_bytes) : "memory");
@@ -1453,7 +1509,8 @@ __global__ void __launch_bounds__(128, D > 128 ? 1 : (MT == 2 ? 2 : 3)) paged_bi
     const float* __restrict__ bias_table, const uint8_t* __restrict__ lut, int lut_n, int nbuckets, T* __restrict__ out,
     int heads, int kv_heads, int dim, int vdim, int ldv, int block_size, int max_blocks, float scale, int sink, int chunk,
     int max_splits, float* __restrict__ part_o, float* __restrict__ part_ml, int mask_block, int wide_weights,
-    const float* __restrict__ sink_vals, const float* __restrict__ slopes, int window, int keep_first) {
+    const float* __restrict__ sink_vals, const float* __restrict__ slopes, int window, int keep_first, float softcap,
+    const T* __restrict__ gate, int64_t ldg) {
   constexpr int BM = 64 * MT;
   constexpr int LDS = D + 8;                    // padded row: 16-byte aligned, conflict-free fragment reads
   constexpr int TILE = MMA_BN * LDS;
@@ -1548,7 +1605,11 @@ __global__ void __launch_bounds__(128, D > 128 ? 1 : (MT == 2 ? 2 : 3)) paged_bi
     m[e] = (sink && chunk == 0) ? sk[e] : -INFINITY;        // log2 domain; with chunks the sink joins in the merge
     l[e] = 0.f;                                 // per-thread partial; the sink's share is added once at the end
   }
-  const float sc2 = scale * LOG2E;
+  // soft-capped scores: cap tanh(scale s / cap) = cap - 2 cap / (1 + e^(2 scale s / cap)), taken once per score tile; what
+  // follows sees them in the log2 domain already
+  const bool capped = softcap > 0.f;
+  const float cap_in = capped ? 2.f * scale * LOG2E / softcap : 0.f, cap_out = softcap * LOG2E;
+  const float sc2 = capped ? 1.f : scale * LOG2E;
   // first / last position any row of this warp sees: tiles beyond are skipped, tiles before need no causal test
   const int wrow0 = row0 + (KS ? 0 : warp * (16 * MT));
   const int koff = KS ? warp * 16 : 0;          // first key of the warp inside a key tile
@@ -1598,6 +1659,15 @@ __global__ void __launch_bounds__(128, D > 128 ? 1 : (MT == 2 ? 2 : 3)) paged_bi
             mma_16816<T>(sacc[mt][nt], qa[mt][1], kb[2], kb[3]);
           }
         }
+      }
+      if (capped) {
+#pragma unroll
+        for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+          for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+            for (int e = 0; e < 4; ++e)
+              sacc[mt][nt][e] = fmaf(-2.f * cap_out, rcpf(1.f + ex2f(sacc[mt][nt][e] * cap_in)), cap_out);
       }
       const int jlast = j0 + koff + NT * 8 - 1;  // last key this warp scores in the tile
       const bool unmasked = jlast <= wlo && (j0 + koff >= wblk || jlast < keep_first);
@@ -1751,6 +1821,7 @@ __global__ void __launch_bounds__(128, D > 128 ? 1 : (MT == 2 ? 2 : 3)) paged_bi
         }
       } else {
         if (sink) lsum += ex2f((sink_vals != nullptr ? sink_vals[g * R + row % R] * LOG2E : 0.f) - mu);
+        osum *= head_gate<T>(gate, ldg, t0 + row / R, g * R + row % R);
         out[unit * vdim + c] = from_f32<T>(lsum > 0.f ? osum / lsum : 0.f);
       }
     }
@@ -1777,7 +1848,7 @@ __global__ void __launch_bounds__(128, D > 128 ? 1 : (MT == 2 ? 2 : 3)) paged_bi
       continue;
     }
     if (sink) l[r] += ex2f(sk[r] - (m[r] == -INFINITY ? 0.f : m[r]));
-    const float inv = l[r] > 0.f ? 1.f / l[r] : 0.f;
+    const float inv = l[r] > 0.f ? head_gate<T>(gate, ldg, t0 + rr[r] / R, g * R + hr[r]) / l[r] : 0.f;
     T* orow = out + unit * vdim;
 #pragma unroll
     for (int nv = 0; nv < D / 8; ++nv) {
@@ -1801,7 +1872,7 @@ __global__ void __launch_bounds__(128) attention_merge_kernel(const float* __res
                                                               int64_t tokens, int heads, int kv_heads, int vdim, int bm,
                                                               int chunk, int max_splits, int sink, int mask_block,
                                                               const float* __restrict__ sink_vals, int window,
-                                                              int keep_first) {
+                                                              int keep_first, const T* __restrict__ gate, int64_t ldg) {
   const int lane = threadIdx.x & 31;
   const int cblocks = (vdim + 31) >> 5;
   const int64_t item = (int64_t)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
@@ -1836,7 +1907,7 @@ __global__ void __launch_bounds__(128) attention_merge_kernel(const float* __res
       if (c < vdim) acc = fmaf(po[(int64_t)(s0 + j) * vdim + c], w, acc);
     }
   }
-  const float inv = l > 0.f ? 1.f / l : 0.f;
+  const float inv = l > 0.f ? head_gate<T>(gate, ldg, tok, (int)(unit % heads)) / l : 0.f;
   if (c < vdim) out[unit * vdim + c] = from_f32<T>(acc * inv);
 }
 
@@ -1847,7 +1918,7 @@ int launch_attention_mma(const void* q, int64_t ldq, const void* k_cache, const 
                          int heads, int kv_heads, int dim, int vdim, int ldv, int block_size, int max_blocks, float scale,
                          int sink, int chunk, int max_splits, float* part_o, float* part_ml, int mask_block,
                          int wide_weights, const float* sink_vals, const float* slopes, int window, int keep_first,
-                         cudaStream_t st) {
+                         float softcap, const void* gate, int64_t ldg, cudaStream_t st) {
   const int R = heads / kv_heads;
   constexpr int BM = 64 * MT;
   const bool kv_same = v_cache == k_cache && ldv == dim;
@@ -1865,13 +1936,13 @@ int launch_attention_mma(const void* q, int64_t ldq, const void* k_cache, const 
   kern<<<grid, 128, smem, st>>>((const T*)q, ldq, (const T*)k_cache, (const T*)v_cache, block_tables, cu_q, ctx_len,
                                 bias_table, lut, lut_n, nbuckets, (T*)out, heads, kv_heads, dim, vdim, ldv, block_size,
                                 max_blocks, scale, sink, chunk, max_splits, part_o, part_ml, mask_block, wide_weights,
-                                sink_vals, slopes, window, keep_first);
+                                sink_vals, slopes, window, keep_first, softcap, (const T*)gate, ldg);
   if (chunk > 0) {
     const int64_t units = tokens * heads * ((vdim + 31) / 32);
     attention_merge_kernel<T><<<(unsigned)((units + 3) / 4), 128, 0, st>>>(part_o, part_ml, token_pos, token_seq, cu_q,
                                                                           (T*)out, tokens, heads, kv_heads, vdim, BM, chunk,
                                                                           max_splits, sink, mask_block, sink_vals, window,
-                                                                          keep_first);
+                                                                          keep_first, (const T*)gate, ldg);
   }
   return CB_LAUNCH_CHECK();
 }
@@ -2319,6 +2390,156 @@ __global__ void __launch_bounds__(256) rotary_kv_write_kernel(T* __restrict__ qk
   }
 }
 
+// ------------------------------------------------------------------------------------------------ convolved q | k | v
+// One warp per (sequence, head, tile of tokens) of projection rows q | k | v: the head's channels pass the causal convolution
+// (window of TAPS - 1 inputs in registers, carried over the tile's tokens); query and key heads are then turned by the token's
+// position and divided by sqrt(mean of squares + eps); queries go to q_out, keys and values into their pages.  fp32 from the
+// first load to the one rounding at the store.  A lane holds VEC adjacent channels per step, ITEMS steps; the head sits in
+// shared memory while it is turned.
+constexpr int CRW_TOK_TILE = 16;
+
+template <typename T> struct ConvRotArgs {
+  const T *x, *w, *state;
+  int64_t ldx;
+  T *q_out, *k_cache, *v_cache;
+  int taps, H, G, dim, vdim, rot, interleaved, unit, block_size, max_blocks;
+  float eps;
+  const float* table;
+  const int *block_tables, *cu_q, *ctx_len, *slots;
+};
+
+template <typename T, int VEC, int ITEMS, int TAPS>
+__global__ void __launch_bounds__(128) conv_rotary_kv_write_kernel(ConvRotArgs<T> a) {
+  struct alignas(sizeof(T) * VEC) Pack { T v[VEC]; };
+  extern __shared__ __align__(16) float crw_smem[];
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int s = blockIdx.z, unit = blockIdx.x * (blockDim.x >> 5) + warp;
+  const int t0 = a.cu_q[s], qlen = a.cu_q[s + 1] - t0;
+  const int j0 = blockIdx.y * CRW_TOK_TILE;
+  if (unit >= a.H + 2 * a.G || j0 >= qlen) return;
+  const bool value = unit >= a.H + a.G;
+  const int width = value ? a.vdim : a.dim;
+  const int c0 = value ? (a.H + a.G) * a.dim + (unit - a.H - a.G) * a.vdim : unit * a.dim;
+  const int C = (a.H + a.G) * a.dim + a.G * a.vdim;
+  const int ctx = a.ctx_len[s];
+  const T* st = a.state + (int64_t)a.slots[s] * (TAPS - 1) * C + c0;
+  const T* xr = a.x + (int64_t)t0 * a.ldx + c0;
+  float wt[ITEMS][TAPS][VEC], win[ITEMS][TAPS > 1 ? TAPS - 1 : 1][VEC];
+#pragma unroll
+  for (int it = 0; it < ITEMS; ++it) {
+    const int c = (lane + 32 * it) * VEC;
+    if (c < width) {
+#pragma unroll
+      for (int i = 0; i < TAPS; ++i)
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) wt[it][i][e] = to_f32<T>(a.w[(int64_t)(c0 + c + e) * TAPS + i]);
+#pragma unroll
+      for (int i = 0; i < TAPS - 1; ++i) {
+        const int rel = j0 - (TAPS - 1) + i;
+        Pack p;
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) p.v[e] = from_f32<T>(0.f);
+        if (rel >= 0) p = *reinterpret_cast<const Pack*>(xr + (int64_t)rel * a.ldx + c);
+        else if (ctx > 0) p = *reinterpret_cast<const Pack*>(st + (int64_t)(TAPS - 1 + rel) * C + c);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) win[it][i][e] = to_f32<T>(p.v[e]);
+      }
+    }
+  }
+  float* sm = crw_smem + warp * (ITEMS * 32 * VEC);
+  const int half = a.rot >> 1;
+  const int j1 = min(j0 + CRW_TOK_TILE, qlen);
+  for (int j = j0; j < j1; ++j) {
+    const int pos = ctx + j;
+    float y[ITEMS][VEC];
+#pragma unroll
+    for (int it = 0; it < ITEMS; ++it) {
+      const int c = (lane + 32 * it) * VEC;
+      if (c < width) {
+        const Pack p = *reinterpret_cast<const Pack*>(xr + (int64_t)j * a.ldx + c);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) {
+          const float cur = to_f32<T>(p.v[e]);
+          float acc = 0.f;
+#pragma unroll
+          for (int i = 0; i < TAPS - 1; ++i) acc = fmaf(wt[it][i][e], win[it][i][e], acc);
+          y[it][e] = fmaf(wt[it][TAPS - 1][e], cur, acc);
+#pragma unroll
+          for (int i = 0; i < TAPS - 2; ++i) win[it][i][e] = win[it][i + 1][e];
+          if (TAPS > 1) win[it][TAPS > 1 ? TAPS - 2 : 0][e] = cur;
+        }
+      }
+    }
+    if (!value && a.rot > 0) {
+      __syncwarp();                                          // the last token's partners have been read
+#pragma unroll
+      for (int it = 0; it < ITEMS; ++it)
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) sm[(lane + 32 * it) * VEC + e] = y[it][e];
+      __syncwarp();
+      const float* cs = a.table + (int64_t)pos * a.rot;
+#pragma unroll
+      for (int it = 0; it < ITEMS; ++it)
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) {
+          const int c = (lane + 32 * it) * VEC + e;
+          if (c < a.rot) {                                   // pair index, partner, and which half of the pair this is
+            const int pi = a.interleaved ? c >> 1 : (c < half ? c : c - half);
+            const int pc = a.interleaved ? c ^ 1 : (c < half ? c + half : c - half);
+            const bool first = a.interleaved ? !(c & 1) : c < half;
+            const float sn = cs[half + pi];
+            y[it][e] = fmaf(y[it][e], cs[pi], first ? -sm[pc] * sn : sm[pc] * sn);
+          }
+        }
+    }
+    if (!value && a.unit) {
+      float ss = 0.f;
+#pragma unroll
+      for (int it = 0; it < ITEMS; ++it)
+        if ((lane + 32 * it) * VEC < width) {
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) ss = fmaf(y[it][e], y[it][e], ss);
+        }
+      const float r = 1.f / sqrtf(warp_sum(ss) / (float)width + a.eps);
+#pragma unroll
+      for (int it = 0; it < ITEMS; ++it)
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) y[it][e] *= r;
+    }
+    T* dst;
+    if (unit < a.H) {
+      dst = a.q_out + ((int64_t)(t0 + j) * a.H + unit) * a.dim;
+    } else {
+      const int64_t row = (int64_t)a.block_tables[(int64_t)s * a.max_blocks + pos / a.block_size] * a.block_size +
+                          pos % a.block_size;
+      dst = value ? a.v_cache + (row * a.G + unit - a.H - a.G) * a.vdim : a.k_cache + (row * a.G + unit - a.H) * a.dim;
+    }
+#pragma unroll
+    for (int it = 0; it < ITEMS; ++it) {
+      const int c = (lane + 32 * it) * VEC;
+      if (c < width) {
+        Pack p;
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) p.v[e] = from_f32<T>(y[it][e]);
+        *reinterpret_cast<Pack*>(dst + c) = p;
+      }
+    }
+  }
+}
+
+template <typename T, int VEC, int ITEMS>
+int launch_conv_rotary(const ConvRotArgs<T>& a, dim3 grid, cudaStream_t st) {
+  const size_t smem = (size_t)4 * ITEMS * 32 * VEC * sizeof(float);
+  switch (a.taps) {
+    case 1: conv_rotary_kv_write_kernel<T, VEC, ITEMS, 1><<<grid, 128, smem, st>>>(a); break;
+    case 2: conv_rotary_kv_write_kernel<T, VEC, ITEMS, 2><<<grid, 128, smem, st>>>(a); break;
+    case 3: conv_rotary_kv_write_kernel<T, VEC, ITEMS, 3><<<grid, 128, smem, st>>>(a); break;
+    case 4: conv_rotary_kv_write_kernel<T, VEC, ITEMS, 4><<<grid, 128, smem, st>>>(a); break;
+    default: return (int)cudaErrorInvalidValue;
+  }
+  return CB_LAUNCH_CHECK();
+}
+
 }  // namespace
 
 // ================================================================================================ C launchers
@@ -2355,6 +2576,7 @@ int64_t cb_state_scan_workspace(int mode, int64_t tokens, int heads, int qk_head
   const int64_t DK = scan_dk(dim), VP = scan_vp(vdim);
   int64_t n = 2 * tokens * qk_heads * DK + tokens * heads * VP;
   if (mode == SCAN_DELTA) n += tokens * heads * DK + (tokens * heads + 3) / 4 * 4;
+  if (mode == SCAN_ROWS) n += tokens * heads * DK;
   if (mode == SCAN_GATED) n += tokens * heads * 4;
   return n;
 }
@@ -2365,19 +2587,21 @@ int cb_state_scan(int mode, const void* q, int64_t ldq, const void* k, int64_t l
                   const int* cu_q, const int* ctx_len, const int* slots, int nseq, int heads, int qk_heads, int dim,
                   int vdim, int act_silu, int unit_qk, float unit_eps, float q_scale, float k_scale,
                   const float* rot_table, int rot_dims, const int* token_pos, int gate_kind, float gate_cap,
-                  float* state_n, float* state_m, int dtype, cudaStream_t st) {
+                  float* state_n, float* state_m, float tau, int dtype, cudaStream_t st) {
   if (nseq == 0 || tokens == 0) return 0;
   if (heads % qk_heads != 0 || rot_dims > dim || (rot_dims & 1)) return (int)cudaErrorInvalidValue;
   if (mode == SCAN_GATED && ((gate_kind != GATE_STEP && gate_kind != GATE_EXP) || araw == nullptr || dt_bias == nullptr ||
                              (gate_kind == GATE_STEP && a_log == nullptr) ||
                              (gate_kind == GATE_EXP && (state_n == nullptr || state_m == nullptr))))
     return (int)cudaErrorInvalidValue;
+  if (mode == SCAN_ROWS && (araw == nullptr || dt_bias == nullptr || !(tau > 0.f))) return (int)cudaErrorInvalidValue;
   ScanParams p{q, k, v, ldq, ldk, ldv, araw, lda, braw, ldb, head_decay, a_log, dt_bias, state, out, cu_q, ctx_len, slots,
                heads, qk_heads, dim, vdim, act_silu, unit_qk, unit_eps, q_scale, k_scale, rot_table, rot_dims, token_pos,
-               gate_kind, gate_cap, state_n, state_m};
+               gate_kind, gate_cap, state_n, state_m, 1.f / tau};
   CB_DISPATCH_FLOAT(dtype, T, {
     if (mode == SCAN_GATED) return launch_scan<SCAN_GATED, T>(p, work, tokens, nseq, st);
     if (mode == SCAN_DELTA) return launch_scan<SCAN_DELTA, T>(p, work, tokens, nseq, st);
+    if (mode == SCAN_ROWS) return launch_scan<SCAN_ROWS, T>(p, work, tokens, nseq, st);
     return launch_scan<SCAN_DECAY, T>(p, work, tokens, nseq, st);
   });
   return CB_LAUNCH_CHECK();
@@ -2560,8 +2784,8 @@ int cb_stream_add_norm(float* x, const void* a0, int64_t ld0, int dt0, const voi
 }
 
 int cb_rotary_half(const void* src, int64_t lds, void* dst, int64_t ldd, int64_t tokens, int heads, int src_hs, int src_off,
-                   int dst_hs, int dst_off, int width, int dims, const float* table, const int* token_pos, int src_dtype,
-                   int dst_dtype, cudaStream_t st) {
+                   int dst_hs, int dst_off, int width, int dims, int interleaved, const float* table, const int* token_pos,
+                   int src_dtype, int dst_dtype, cudaStream_t st) {
   if (tokens == 0 || heads == 0 || width == 0) return 0;
   if (dims > width || (dims & 1) || src_dtype != dst_dtype) return (int)cudaErrorInvalidValue;
   CB_DISPATCH_FLOAT(src_dtype, T, {
@@ -2574,22 +2798,22 @@ int cb_rotary_half(const void* src, int64_t lds, void* dst, int64_t ldd, int64_t
     const unsigned grid = (unsigned)((total + 255) / 256 < 148 * 32 ? (total + 255) / 256 : 148 * 32);
     if (vec)
       rotary_half_kernel<T, V><<<grid, 256, 0, st>>>((const T*)src, lds, (T*)dst, ldd, tokens, heads, src_hs, src_off,
-                                                     dst_hs, dst_off, width, dims, table, token_pos);
+                                                     dst_hs, dst_off, width, dims, interleaved, table, token_pos);
     else
       rotary_half_kernel<T, 1><<<grid, 256, 0, st>>>((const T*)src, lds, (T*)dst, ldd, tokens, heads, src_hs, src_off,
-                                                     dst_hs, dst_off, width, dims, table, token_pos);
+                                                     dst_hs, dst_off, width, dims, interleaved, table, token_pos);
   });
   return CB_LAUNCH_CHECK();
 }
 
-int cb_latent_kv_write(const void* z, int64_t ldz, const void* w, int w_dtype, float eps, int rank, int rot,
+int cb_latent_kv_write(const void* z, int64_t ldz, const void* w, int w_dtype, float eps, int rank, int rot, int interleaved,
                        const float* table, void* cache, const int* block_tables, const int* token_seq, const int* token_pos,
                        int64_t tokens, int block_size, int max_blocks, int dtype, cudaStream_t st) {
   if (tokens == 0) return 0;
   if (rot & 1) return (int)cudaErrorInvalidValue;
   const unsigned grid = (unsigned)((tokens + 7) / 8);
 #define CB_LATENT_WRITE(T, TW, V)                                                                                     \
-  latent_kv_write_kernel<T, TW, V><<<grid, 256, 0, st>>>((const T*)z, ldz, (const TW*)w, eps, rank, rot, table,        \
+  latent_kv_write_kernel<T, TW, V><<<grid, 256, 0, st>>>((const T*)z, ldz, (const TW*)w, eps, rank, rot, interleaved, table, \
                                                          (T*)cache, block_tables, token_seq, token_pos, tokens,       \
                                                          block_size, max_blocks)
   CB_DISPATCH_FLOAT(dtype, T, {
@@ -2639,7 +2863,8 @@ int cb_paged_bias_attention(const void* q, int64_t ldq, const void* k_cache, con
                             const int* token_seq, const int* token_pos, const float* bias_table, const int* bucket_start,
                             int nbuckets, void* out, int64_t tokens, int heads, int kv_heads, int dim, int vdim, int ldv,
                             int block_size, int max_blocks, float scale, int sink, int mask_block, const float* sink_vals,
-                            const float* slopes, int window, int keep_first, int dtype, cudaStream_t st) {
+                            const float* slopes, int window, int keep_first, float softcap, const void* gate, int64_t ldg,
+                            int dtype, cudaStream_t st) {
   if (tokens == 0) return 0;
   if (vdim > 32 * ATT_MAX_VREG || heads % kv_heads != 0) return (int)cudaErrorInvalidValue;
   const int nwarps = 4;
@@ -2649,7 +2874,7 @@ int cb_paged_bias_attention(const void* q, int64_t ldq, const void* k_cache, con
     paged_bias_attention_kernel<T><<<(unsigned)((units + nwarps - 1) / nwarps), nwarps * 32, smem, st>>>(
         (const T*)q, ldq, (const T*)k_cache, (const T*)v_cache, block_tables, token_seq, token_pos, bias_table,
         bucket_start, nbuckets, (T*)out, tokens, heads, kv_heads, dim, vdim, ldv, block_size, max_blocks, scale, sink,
-        mask_block, sink_vals, slopes, window, keep_first);
+        mask_block, sink_vals, slopes, window, keep_first, softcap, (const T*)gate, ldg);
   });
   return CB_LAUNCH_CHECK();
 }
@@ -2662,7 +2887,8 @@ int cb_paged_bias_attention_mma(const void* q, int64_t ldq, const void* k_cache,
                                 int nbuckets, void* out, int64_t tokens, int nseq, int max_q, int heads, int kv_heads, int dim, int vdim, int ldv,
                                 int block_size, int max_blocks, float scale, int sink, int chunk, int max_splits,
                                 float* part_o, float* part_ml, int mask_block, int wide_weights, const float* sink_vals,
-                                const float* slopes, int window, int keep_first, int dtype, cudaStream_t st) {
+                                const float* slopes, int window, int keep_first, float softcap, const void* gate,
+                                int64_t ldg, int dtype, cudaStream_t st) {
   if (nseq == 0 || max_q == 0) return 0;
   if (heads % kv_heads != 0 || dim % 8 != 0 || vdim % 8 != 0 || dim > 256 || vdim > 256 || (ldq & 7) || ((uintptr_t)q & 15) ||
       (ldv & 7) || ldv < vdim ||
@@ -2674,7 +2900,7 @@ int cb_paged_bias_attention_mma(const void* q, int64_t ldq, const void* k_cache,
 #define CB_ATT_ARGS                                                                                                   \
   q, ldq, k_cache, v_cache, block_tables, cu_q, ctx_len, token_pos, token_seq, bias_table, lut, lut_n, nbuckets, out,  \
       tokens, nseq, max_q, heads, kv_heads, dim, vdim, ldv, block_size, max_blocks, scale, sink, chunk, max_splits,    \
-      part_o, part_ml, mask_block, wide_weights, sink_vals, slopes, window, keep_first, st
+      part_o, part_ml, mask_block, wide_weights, sink_vals, slopes, window, keep_first, softcap, gate, ldg, st
 #define CB_ATT_MMA(T, D)                                                                                              \
   if (few) return launch_attention_mma<T, D, 1, true>(CB_ATT_ARGS);                                                   \
   if (wide) return launch_attention_mma<T, D, 2>(CB_ATT_ARGS);                                                        \
@@ -2840,6 +3066,34 @@ int cb_rotary_kv_write(void* qkv, int64_t ld, int64_t tokens, int H, int G, int 
       rotary_kv_write_kernel<T, 1><<<grid, 256, 0, st>>>((T*)qkv, ld, tokens, H, G, dim, vdim, rot, table, (T*)k_cache,
                                                          (T*)v_cache, block_tables, token_seq, token_pos, block_size,
                                                          max_blocks, per);
+  });
+  return CB_LAUNCH_CHECK();
+}
+
+// q | k | v projection rows through the convolution (1 to 4 taps), rotary positions and the unit norm into q_out / the pages.
+// `vec`: heads up to 256 wide whose widths, strides and addresses allow four channels per access; else heads up to 128 wide.
+int cb_conv_rotary_kv_write(const void* x, int64_t ldx, const void* w, void* state, int taps, void* q_out, int H, int G, int dim,
+                            int vdim, int rot, int interleaved, const float* table, int unit, float eps, void* k_cache,
+                            void* v_cache, const int* block_tables, const int* cu_q, const int* ctx_len, const int* slots,
+                            int nseq, int max_q, int block_size, int max_blocks, int vec, int dtype, cudaStream_t st) {
+  if (nseq == 0 || max_q == 0) return 0;
+  const int width = dim > vdim ? dim : vdim, C = (H + G) * dim + G * vdim;
+  if (taps < 1 || taps > 4 || rot > dim || (rot & 1) || (rot > 0 && table == nullptr) || width > (vec ? 256 : 128))
+    return (int)cudaErrorInvalidValue;
+  CB_DISPATCH_FLOAT(dtype, T, {
+    const uintptr_t al = 4 * sizeof(T) - 1;
+    if (vec && (dim % 4 || vdim % 4 || ldx % 4 || ((uintptr_t)x & al) || ((uintptr_t)q_out & al) || ((uintptr_t)k_cache & al) ||
+                ((uintptr_t)v_cache & al) || ((uintptr_t)state & al)))
+      return (int)cudaErrorInvalidValue;
+    const ConvRotArgs<T> a{(const T*)x, (const T*)w, (const T*)state, ldx, (T*)q_out, (T*)k_cache, (T*)v_cache, taps, H, G, dim,
+                           vdim, rot, interleaved, unit, block_size, max_blocks, eps, table, block_tables, cu_q, ctx_len, slots};
+    const dim3 grid((H + 2 * G + 3) / 4, (max_q + CRW_TOK_TILE - 1) / CRW_TOK_TILE, nseq);
+    const int rc = !vec ? launch_conv_rotary<T, 1, 4>(a, grid, st)
+                        : (width <= 128 ? launch_conv_rotary<T, 4, 1>(a, grid, st) : launch_conv_rotary<T, 4, 2>(a, grid, st));
+    if (rc != 0) return rc;
+    if (taps > 1)
+      short_conv_state_kernel<T><<<dim3((C + 127) / 128, nseq), 128, 0, st>>>((const T*)x, ldx, (T*)state, cu_q, ctx_len, slots,
+                                                                             C, taps);
   });
   return CB_LAUNCH_CHECK();
 }

@@ -63,16 +63,21 @@ class MixerSpec:
     kind "delta":      gated delta rule with ONE decay per head, exp(-exp(A_log) softplus(W_a h + dt_bias)), a write
                        strength sigmoid(W_b h), short causal convolutions of `conv` taps + silu on q, k, v, unit-length
                        q / k, the read-out brought to unit RMS per head, weighted and gated by silu(W_g h).
+    kind "gla":        gated linear attention: an outer-product memory per head whose ROWS decay by sigmoid(z)^(1 / `tau`),
+                       z per head and key channel from a low-rank projection (`decay_rank`) plus a bias, q scaled by
+                       dim^-1/2, the read-out brought to unit RMS per head, weighted and gated by silu(W_g h).
 
     kind "latent" also takes: `q_rank` (queries through an RMS-normalised latent of that width), `window`,
-    `sink_learned`, `rot_scaling`.
+    `sink_learned`, `rot_scaling`, `rot_interleaved`, `head_gate`.
 
     kind "attention" also takes: rotary positions on the first `rot_dims` channels of every q / k head (pairs (2i, 2i + 1)
     when `rot_interleaved`, else (i, i + rot_dims / 2)); `head_unit_norm` (q and k divided by their root mean square over
     the head, after the rotation, no weight); `mask_block` (a position sees only the keys of its own block of that many
     positions, counted from the start of the sequence); `out_gate` (heads times sigmoid(W_g x) before the output
-    projection); `conv` (a causal convolution of that many taps on every channel of the q and k projections, no
-    activation; its last inputs are carried like a recurrent state); `head_norm` (RMS norm of every q / k head with one
+    projection); `head_gate` (the same with ONE number per head); `softcap` (score <- softcap x tanh(score / softcap), before
+    mask and sink); `conv` (a causal convolution of that many taps on every channel of the q and k projections, no
+    activation; its last inputs are carried like a recurrent state; with `conv_values` on the v projection too, and rotary
+    positions / `head_unit_norm` may follow it); `head_norm` (RMS norm of every q / k head with one
     weight over the head's channels per projection); `values_from_keys` (no value projection: the values are the keys as
     they leave the convolution, before any norm); `dist_slopes` (score minus 2^(-8 (h + 1) / heads) x distance);
     `window` (a position sees itself and the window - 1 positions before it), `keep_first` (with a window: the first that
@@ -115,9 +120,14 @@ class MixerSpec:
     q_rank: int = 0                   # latent: width of the normalised query latent (0 = queries straight from the input)
     window: int = 0                   # attention / latent: > 0 keeps the keys pos - window + 1 .. pos
     sink_learned: bool = False        # the softmax sink's score is a learned number per head (implies a sink)
+    softcap: float = 0.0              # attention: score <- softcap * tanh(score / softcap) (0 = none)
+    head_gate: bool = False           # attention / latent: head h's output * sigmoid(W_g x)_h, one number per head
+    conv_values: bool = False         # attention: the convolution also covers the value projection
+    tau: float = 1.0                  # gla: row decay = sigmoid(z)^(1 / tau)
     keep_first: int = 0               # attention: keys 0 .. keep_first - 1 stay visible beside the window
-    rot_scaling: Optional[List[float]] = None     # (factor, original length, fast, slow): stretched slow frequencies;
-                                                  # (factor,): every frequency divided by it
+    rot_scaling: Optional[List[Any]] = None       # (factor, original length, fast, slow): stretched slow frequencies;
+                                                  # (factor,): every frequency divided by it;
+                                                  # ("wavelength", factor, low, high, original length): by wavelength
     head_norm: bool = False           # attention: RMS norm per q / k head with a weight shared by the heads
     values_from_keys: bool = False    # attention: values = keys before their norm (no value projection)
     dist_slopes: bool = False         # attention: score -= 2^(-8 (h + 1) / heads) * (query position - key position)
@@ -131,8 +141,7 @@ class MixerSpec:
         assert self.heads % self.kv_heads == 0, "query heads must be a multiple of key/value heads"
         if self.parts is not None:
             self.parts = [MixerSpec(**p) if isinstance(p, dict) else p for p in self.parts]
-            assert sum(p.paged for p in self.parts) <= 1 and sum(p.recurrent for p in self.parts) <= 1, \
-                "a pair holds at most one paged and one recurrent mixer (they share the layer's pages / state slot)"
+            assert sum(p.paged for p in self.parts) <= 1, "a pair holds at most one paged mixer (the layer's pages are its own)"
 
     @property
     def recurrent(self) -> bool:
@@ -140,7 +149,7 @@ class MixerSpec:
             return any(p.recurrent for p in self.parts)
         if self.kind == "attention":                  # a convolution in front of attention carries its last inputs
             return self.conv > 0
-        return self.kind in ("lightning", "channel_delta", "retention", "mlstm", "ssd", "rglru", "delta")
+        return self.kind in ("lightning", "channel_delta", "retention", "mlstm", "ssd", "rglru", "delta", "gla")
 
     @property
     def paged(self) -> bool:
@@ -156,10 +165,13 @@ class MixerSpec:
         return self if self.paged else None
 
     @property
-    def recurrent_part(self) -> Optional["MixerSpec"]:
-        if self.kind == "pair":
-            return next((p for p in self.parts if p.recurrent), None)
-        return self if self.recurrent else None
+    def recurrent_parts(self) -> List[Tuple[str, "MixerSpec"]]:
+        """(tag, mixer) of every mixer that keeps state in the layer's slot.  The tag is appended to the names of the
+        mixer's state tensors: empty, except where several parts of a pair keep state (".0", ".1", .. by part)."""
+        if self.kind != "pair":
+            return [("", self)] if self.recurrent else []
+        parts = [(j, p) for j, p in enumerate(self.parts) if p.recurrent]
+        return [(f".{j}" if len(parts) > 1 else "", p) for j, p in parts]
 
 
 @dataclass
@@ -205,7 +217,9 @@ class LayerSpec:
     ff: Optional[int] = None          # dense feed-forward width; None = no dense feed-forward
     moe: Optional[ExpertFFSpec] = None  # routed feed-forward instead of a dense one
     ff_act: Optional[str] = None      # dense feed-forward: activation of this layer instead of `ModelConfig.hidden_act`
-                                      # ("polynorm": learned mix of the first three powers, each brought to unit RMS)
+                                      # ("polynorm": learned mix of the first three powers, each brought to unit RMS;
+                                      # "clamped": gated unit of `ExpertFFSpec`, clamped at `ff_limit`)
+    ff_limit: float = 7.0             # "clamped" dense feed-forward: the clamp
 
     def __post_init__(self) -> None:
         if isinstance(self.mixer, dict):

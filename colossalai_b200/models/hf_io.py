@@ -49,6 +49,10 @@ def config_from_hf(hf: dict) -> ModelConfig:
         from .sodurax import sodurax_config
 
         return sodurax_config(hf)
+    if hf.get("architecture") == "Sumolorn":
+        from .sumolorn import sumolorn_config
+
+        return sumolorn_config(hf)
     if mt == "gpt2":
         return ModelConfig(model_type="gpt2", vocab_size=hf["vocab_size"], hidden_size=hf["n_embd"],
                            intermediate_size=hf.get("n_inner") or 4 * hf["n_embd"], num_hidden_layers=hf["n_layer"],
@@ -512,6 +516,10 @@ def load_hf_checkpoint(path: str, dtype: torch.dtype = torch.bfloat16, device: s
         from .sodurax import load_sodurax
 
         return load_sodurax(path, hf_cfg, dtype, device)
+    if hf_cfg.get("architecture") == "Sumolorn":
+        from .sumolorn import load_sumolorn
+
+        return load_sumolorn(path, hf_cfg, dtype, device)
     cfg = config_from_hf(hf_cfg)
     model = build_model(cfg).to(dtype)
     merged: Dict[str, torch.Tensor] = {}

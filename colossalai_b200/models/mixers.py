@@ -12,13 +12,14 @@
   * `SelectiveStateSpace`: state space with input-dependent step sizes behind a causal convolution, gate before the norm;
   * `GatedLinearRecurrence`: per-channel real-gated linear recurrent unit behind a causal convolution, times a GELU branch;
   * `MixerPair`: mixers side by side on the same input; their RMS-normed outputs are averaged;
-  * `DeltaMixer`: gated delta rule with one decay per head behind short causal convolutions, gated unit-RMS read-out.
+  * `DeltaMixer`: gated delta rule with one decay per head behind short causal convolutions, gated unit-RMS read-out;
+  * `GatedLinearAttention`: outer-product memory whose rows decay per token, head and key channel, gated unit-RMS read-out.
 
 `BiasSinkAttention` also covers plain paged softmax attention with rotary positions (half or interleaved pairs, on a part
 of the head), a weightless unit norm of q / k heads, a block mask (a position sees its own block of positions only), a
-sigmoid output gate, a short convolution on q | k, an RMS norm per q / k head with a shared weight, values taken from the
-keys, a linear distance penalty per head, a sliding window (also with the first keys kept) and a learned sink score: every one of these is a field of the
-`MixerSpec`.
+sigmoid output gate (per channel or per head), a short convolution on q | k or q | k | v, an RMS norm per q / k head with a
+shared weight, values taken from the keys, a linear distance penalty per head, soft-capped scores, a sliding window (also with
+the first keys kept) and a learned sink score: every one of these is a field of the `MixerSpec`.
 
 Every mixer keeps the call signature of `Attention` (`forward(x, meta, rope, kv_cache)`) and is selected per layer by
 `ModelConfig.layer_specs[i].mixer.kind` (`build_mixer`).  `kv_cache` is the step runtime (`inference.modeling.PagedKVRuntime`):
@@ -38,7 +39,13 @@ from ..ops import mixers as mops
 from .config import MixerSpec, ModelConfig
 
 __all__ = ["BiasSinkAttention", "LightningAttention", "ChannelDeltaMixer", "LatentAttention", "Retention", "MatrixLSTM",
-           "SelectiveStateSpace", "GatedLinearRecurrence", "MixerPair", "DeltaMixer", "build_mixer"]
+           "SelectiveStateSpace", "GatedLinearRecurrence", "MixerPair", "DeltaMixer", "GatedLinearAttention", "build_mixer"]
+
+
+def _pad8(rows: int) -> int:
+    """Output rows of a stacked projection, rounded up so that token rows of 16-bit results start on 16-byte boundaries (the
+    vector and tensor-core paths of the kernels behind it); the rows added carry zero weights."""
+    return (rows + 7) // 8 * 8
 
 
 class _MixerBase(nn.Module):
@@ -46,7 +53,13 @@ class _MixerBase(nn.Module):
         super().__init__()
         self.cfg, self.spec, self.layer_idx = cfg, spec, layer_idx
         self.shard_config = None
+        self.state_tag = ""                 # set by a pair several parts of which keep state in the layer's slot
         self._aux_cache: Dict[Tuple[str, str], torch.Tensor] = {}
+
+    def _state(self, kv_cache) -> Dict[str, torch.Tensor]:
+        """This mixer's state tensors of the layer's current run."""
+        st, tag = kv_cache.layer_state(self.layer_idx), self.state_tag
+        return {n[: -len(tag)]: t for n, t in st.items() if n.endswith(tag)} if tag else st
 
     def _aux(self, name: str, device, make) -> torch.Tensor:
         """Small constant tensors in exact fp32 / int32 on the compute device (built once per device)."""
@@ -66,15 +79,18 @@ class BiasSinkAttention(_MixerBase):
         H, G, d, dv = spec.heads, spec.kv_heads, spec.dim, spec.vdim
         assert spec.rot_dims % 2 == 0 and spec.rot_dims <= d
         assert not spec.values_from_keys or (dv == d and not spec.v_mix), "values taken from the keys are key-wide"
-        assert not (spec.conv and (spec.rot_dims or spec.head_unit_norm or spec.proj_norm)), \
+        assert not (spec.conv and not spec.conv_values and (spec.rot_dims or spec.head_unit_norm or spec.proj_norm)), \
             "the convolution on q | k is followed by the per-head norm only"
+        assert not (spec.conv_values and (spec.head_norm or spec.proj_norm or spec.values_from_keys or spec.v_mix)), \
+            "the convolution on q | k | v is followed by rotary positions and the unit norm only"
         assert not (spec.keep_first and not (spec.window or spec.mask_block)), "kept first keys go with a window"
         # q | k | v (| output gate): one GEMM reads the layer input (no v with `values_from_keys`)
         self.v_width = 0 if spec.values_from_keys else G * dv
-        self.qkv_proj = nn.Linear(cfg.hidden_size, H * d + G * d + self.v_width + (H * dv if spec.out_gate else 0),
-                                  bias=spec.bias)
-        if spec.conv:
-            self.conv_weight = nn.Parameter(torch.zeros((H + G) * d, spec.conv))       # q channels, then k channels
+        self.gate_width = H * dv if spec.out_gate else (H if spec.head_gate else 0)
+        rows = H * d + G * d + self.v_width + self.gate_width
+        self.qkv_proj = nn.Linear(cfg.hidden_size, _pad8(rows) if spec.head_gate else rows, bias=spec.bias)
+        if spec.conv:                       # q channels, then k channels, then (`conv_values`) v channels
+            self.conv_weight = nn.Parameter(torch.zeros((H + G) * d + (self.v_width if spec.conv_values else 0), spec.conv))
         if spec.head_norm:
             self.q_head_norm_weight = nn.Parameter(torch.ones(d))
             self.k_head_norm_weight = nn.Parameter(torch.ones(d))
@@ -94,10 +110,21 @@ class BiasSinkAttention(_MixerBase):
         sp, eps = self.spec, self.cfg.norm_eps
         H, G, d, dv = sp.heads, sp.kv_heads, sp.dim, sp.vdim
         qkv = self.qkv_proj(x)
-        q, k, v, gate = qkv.split([H * d, G * d, self.v_width, H * dv if sp.out_gate else 0], dim=-1)
-        if sp.conv:
+        a, b = H * d, (H + G) * d
+        q, k, v = qkv[:, :a], qkv[:, a:b], qkv[:, b: b + self.v_width]
+        gate = qkv[:, b + self.v_width: b + self.v_width + self.gate_width]
+        if sp.conv and sp.conv_values:
+            # one pass over q | k | v: convolution, rotary positions, unit norm of the q / k heads, page write
+            kc, vc = kv_cache.pages(self.layer_idx)
+            table = mops.rotary_table(kv_cache.max_len_host, sp.rot_dims, sp.rot_base, x.device, sp.rot_scaling) \
+                if sp.rot_dims else None
+            q = mops.conv_rotary_kv_write(qkv[:, : b + self.v_width], self.conv_weight, self._state(kv_cache)["conv"], H, G, d,
+                                          dv, sp.rot_dims, sp.rot_interleaved, table, eps if sp.head_unit_norm else None, kc,
+                                          vc, kv_cache.block_tables, kv_cache.ragged)
+            k = v = None
+        elif sp.conv:
             # the convolution comes directly after the projection; its window of last inputs lives in the layer's slot
-            qk = mops.short_conv_silu(qkv[:, : (H + G) * d], self.conv_weight, kv_cache.layer_state(self.layer_idx)["conv"],
+            qk = mops.short_conv_silu(qkv[:, : (H + G) * d], self.conv_weight, self._state(kv_cache)["conv"],
                                       kv_cache.ragged, activation=False)
             q, k = qk[:, : H * d], qk[:, H * d:]
         if sp.values_from_keys:
@@ -120,7 +147,7 @@ class BiasSinkAttention(_MixerBase):
                 if sp.rot_dims else None
             mops.rotary_kv_write(qkv, H, G, d, dv, sp.rot_dims, table, kc, vc, kv_cache.block_tables, kv_cache.ragged)
             k = v = None
-        elif sp.rot_dims or sp.head_unit_norm:
+        elif (sp.rot_dims or sp.head_unit_norm) and not sp.conv:
             # q and k heads sit side by side in the projection: rotated and normalised in place, in one launch
             table = mops.rotary_table(kv_cache.max_len_host, sp.rot_dims, sp.rot_base, x.device, sp.rot_scaling) \
                 if sp.rot_dims else None
@@ -149,7 +176,8 @@ class BiasSinkAttention(_MixerBase):
         o = kv_cache.attend_ragged(self.layer_idx, q, k, v, self.scale, bias_table=table, bucket_starts=starts,
                                    sink=sp.sink or sp.sink_learned, v_other=v_other, lam=lam, lut=lut,
                                    mask_block=sp.mask_block, wide_weights=sp.wide_weights, sink_values=sinks,
-                                   slopes=slopes, window=sp.window, keep_first=sp.keep_first)
+                                   slopes=slopes, window=sp.window, keep_first=sp.keep_first, softcap=sp.softcap,
+                                   head_gate=gate if sp.head_gate else None)
         if sp.out_gate:
             o = mops.sigmoid_gate_mul(o, gate)
         return self.o_proj(o)
@@ -170,7 +198,7 @@ class LightningAttention(_MixerBase):
         z = self.in_proj(x)
         q, k, v, g = z.split([H * d, H * d, H * dv, H * dv], dim=-1)
         decay = self._aux("decay", x.device, lambda: torch.tensor(sp.decay, dtype=torch.float64).float())
-        st = kv_cache.layer_state(self.layer_idx)
+        st = self._state(kv_cache)
         o = mops.state_scan_decay(q, k, v, decay, st["S"], kv_cache.ragged, H, d, dv, act_silu=True)
         o = mops.gated_group_rms_norm(o, self.norm_weight, g, H * dv, self.cfg.norm_eps, x.dtype)
         return self.o_proj(o)
@@ -196,7 +224,7 @@ class ChannelDeltaMixer(_MixerBase):
         H, G, d, dv = sp.heads, sp.kv_heads, sp.dim, sp.vdim
         z = self.in_proj(x)
         qkv, b, a1, g1 = z.split([self.conv_channels, H, sp.decay_rank, sp.gate_rank], dim=-1)
-        st = kv_cache.layer_state(self.layer_idx)
+        st = self._state(kv_cache)
         ragged = kv_cache.ragged
         qkv = mops.short_conv_silu(qkv, self.conv_weight, st["conv"], ragged)
         q, k, v = qkv.split([G * d, G * d, H * dv], dim=-1)
@@ -233,7 +261,7 @@ class DeltaMixer(_MixerBase):
         H, G, d, dv = sp.heads, sp.kv_heads, sp.dim, sp.vdim
         z = self.in_proj(x)
         qkv, b, a, gate = z.split([self.conv_channels, H, H, H * dv], dim=-1)
-        st = kv_cache.layer_state(self.layer_idx)
+        st = self._state(kv_cache)
         ragged = kv_cache.ragged
         qkv = mops.short_conv_silu(qkv, self.conv_weight, st["conv"], ragged)
         q, k, v = qkv.split([G * d, G * d, H * dv], dim=-1)
@@ -258,14 +286,17 @@ class LatentAttention(_MixerBase):
     Options of the spec: `q_rank` > 0 - the queries come through a latent of their own, q = W_uq (rms(W_dq h) w_dq) (the
     down-projection shares the GEMM that reads the layer input); `window` - a position sees the last `window` positions;
     `sink_learned` - a learned score per head joins the softmax's denominator; `rot_scaling` - stretched rotary
-    frequencies (`ops.mixers.rotary_frequencies`)."""
+    frequencies (`ops.mixers.rotary_frequencies`); `rot_interleaved` - rotary pairs are neighbours; `head_gate` - head n's
+    result times sigmoid(W_g h)_n, applied in the latent space (one number per head commutes with V_n), its rows share the
+    GEMM that reads the layer input."""
 
     def __init__(self, cfg: ModelConfig, spec: MixerSpec, layer_idx: int) -> None:
         super().__init__(cfg, spec, layer_idx)
         H, d, r, dv, R = spec.heads, spec.dim, spec.rot_dim, spec.vdim, spec.kv_rank
         assert spec.rot_dims in (0, r) and r % 2 == 0, "the decoupled key part is rotated as a whole"
         self.q_width = spec.q_rank or H * (d + r)
-        self.in_proj = nn.Linear(cfg.hidden_size, self.q_width + R + r, bias=False)      # q (or its latent) | latent | key part
+        rows = self.q_width + R + r                                # q (or its latent) | latent | key part (| gates)
+        self.in_proj = nn.Linear(cfg.hidden_size, _pad8(rows + H) if spec.head_gate else rows, bias=False)
         if spec.q_rank:
             self.dq_norm_weight = nn.Parameter(torch.ones(spec.q_rank))
             self.uq_proj = nn.Linear(spec.q_rank, H * (d + r), bias=False)
@@ -284,23 +315,25 @@ class LatentAttention(_MixerBase):
         H, d, r, dv, R = sp.heads, sp.dim, sp.rot_dim, sp.vdim, sp.kv_rank
         T = x.shape[0]
         z = self.in_proj(x)
-        q, dkv = z[:, : self.q_width], z[:, self.q_width:]
+        c0, c1 = self.q_width, self.q_width + R + r
+        q, dkv = z[:, :c0], z[:, c0:c1]
         if sp.q_rank:
             q = self.uq_proj(mops.head_rms_norm(q, 1, 0, sp.q_rank, self.dq_norm_weight, None, self.cfg.norm_eps))
         ragged = kv_cache.ragged
         table = mops.rotary_table(kv_cache.max_len_host, r, sp.rot_base, x.device, sp.rot_scaling)
         mops.latent_kv_write(dkv, self.dkv_norm_weight, self.cfg.norm_eps, R, table, kv_cache.latent_cache(self.layer_idx),
-                             kv_cache.block_tables, ragged)
+                             kv_cache.block_tables, ragged, interleaved=sp.rot_interleaved)
         qa = torch.empty(T, H * (R + r), dtype=x.dtype, device=x.device)
         qa3 = qa.view(T, H, R + r)
         torch.bmm(q.view(T, H, d + r)[..., :d].transpose(0, 1), self.uk, out=qa3[..., :R].transpose(0, 1))
-        mops.rotary_half(q, qa, H, d + r, d, R + r, R, r, r, table, ragged.token_pos)
+        mops.rotary_half(q, qa, H, d + r, d, R + r, R, r, r, table, ragged.token_pos, interleaved=sp.rot_interleaved)
         sinks = self._aux("sink", x.device, lambda: self.sink_logit.detach().float()) if sp.sink_learned else None
         o = kv_cache.attend_latent(self.layer_idx, qa, self.scale, R, window=sp.window,
-                                   sink=sp.sink or sp.sink_learned, sink_values=sinks,
-                                   wide_weights=sp.wide_weights)                              # [T, H x R]
-        o = torch.bmm(o.view(T, H, R).transpose(0, 1), self.uv.transpose(1, 2))        # [H, T, dv]
-        return self.o_proj(o.transpose(0, 1).reshape(T, H * dv))
+                                   sink=sp.sink or sp.sink_learned, sink_values=sinks, wide_weights=sp.wide_weights,
+                                   head_gate=z[:, c1:c1 + H] if sp.head_gate else None)       # [T, H x R]
+        y = torch.empty(T, H * dv, dtype=x.dtype, device=x.device)
+        torch.bmm(o.view(T, H, R).transpose(0, 1), self.uv.transpose(1, 2), out=y.view(T, H, dv).transpose(0, 1))
+        return self.o_proj(y)
 
 
 class Retention(_MixerBase):
@@ -324,7 +357,7 @@ class Retention(_MixerBase):
         q, k, v, g = z.split([H * d, H * d, H * dv, H * dv], dim=-1)
         decay = self._aux("decay", x.device, lambda: torch.tensor(sp.decay, dtype=torch.float64).float())
         table = mops.rotary_table(kv_cache.max_len_host, sp.rot_dims, sp.rot_base, x.device) if sp.rot_dims else None
-        st = kv_cache.layer_state(self.layer_idx)
+        st = self._state(kv_cache)
         o = mops.state_scan_decay(q, k, v, decay, st["S"], kv_cache.ragged, H, d, dv, act_silu=False, rot_table=table,
                                   rot_dims=sp.rot_dims, k_scale=d ** -0.5)
         o = mops.gated_group_rms_norm(o, None, g, dv, self.cfg.norm_eps, x.dtype, gate_act="silu")
@@ -352,7 +385,7 @@ class MatrixLSTM(_MixerBase):
         z = self.in_proj(x)
         q, k, v, g, gates = z.split([H * d, H * d, H * dv, H * dv, 2 * H], dim=-1)
         bias = self._aux("gate_bias", x.device, lambda: self.gate_bias.detach().float())
-        st = kv_cache.layer_state(self.layer_idx)
+        st = self._state(kv_cache)
         o = mops.state_scan_mlstm(q, k, v, gates, bias, sp.gate_cap, st["S"], st["n"], st["m"], kv_cache.ragged, H, d, dv,
                                   q_scale=d ** -0.5)
         o = mops.gated_group_rms_norm(o, self.norm_weight, g, dv, self.cfg.norm_eps, x.dtype)
@@ -385,7 +418,7 @@ class SelectiveStateSpace(_MixerBase):
         H, dv, N, G = sp.heads, sp.vdim, sp.state, sp.groups
         zz = self.in_proj(x)
         z, xbc, dt = zz.split([self.inner, self.conv_channels, H], dim=-1)
-        st = kv_cache.layer_state(self.layer_idx)
+        st = self._state(kv_cache)
         ragged = kv_cache.ragged
         xbc = mops.short_conv_silu(xbc, self.conv_weight, st["conv"], ragged, bias=self.conv_bias)
         xs, b, c = xbc.split([self.inner, G * N, G * N], dim=-1)
@@ -423,7 +456,7 @@ class GatedLinearRecurrence(_MixerBase):
         T = x.shape[0]
         z = self.in_proj(x)
         branch, xb = z[:, :C], z[:, C:]
-        st = kv_cache.layer_state(self.layer_idx)
+        st = self._state(kv_cache)
         ragged = kv_cache.ragged
         u = mops.short_conv_silu(xb, self.conv_weight, st["conv"], ragged, activation=False, bias=self.conv_bias)
         ub = u.view(T, nb, C // nb).transpose(0, 1)                                      # [blocks, T, bw]
@@ -437,16 +470,46 @@ class GatedLinearRecurrence(_MixerBase):
         return self.o_proj(s)
 
 
+class GatedLinearAttention(_MixerBase):
+    """W_in h = [q | k | v | gate | a]; z = W_up a + bias (W_up's products keep their fp32 accumulators).  Per head a matrix
+    S [dim, vdim], zero at the start of a sequence and carried in fp32: S <- diag(sigmoid(z)^(1 / tau)) S + outer(k, v),
+    o = S^T q with q scaled by dim^-1/2.  Every head's o is divided by its root mean square, multiplied by a weight over
+    vdim that the heads share and by silu(gate), and projected."""
+
+    def __init__(self, cfg: ModelConfig, spec: MixerSpec, layer_idx: int) -> None:
+        super().__init__(cfg, spec, layer_idx)
+        H, d, dv = spec.heads, spec.dim, spec.vdim
+        self.in_proj = nn.Linear(cfg.hidden_size, _pad8(2 * H * d + 2 * H * dv + spec.decay_rank), bias=False)
+        self.decay_up = nn.Linear(spec.decay_rank, H * d, bias=False)
+        self.decay_bias = nn.Parameter(torch.zeros(H * d))
+        self.norm_weight = nn.Parameter(torch.ones(dv))
+        self.o_proj = nn.Linear(H * dv, cfg.hidden_size, bias=False)
+
+    def forward(self, x: torch.Tensor, meta, rope=None, kv_cache=None) -> torch.Tensor:
+        sp = self.spec
+        H, d, dv = sp.heads, sp.dim, sp.vdim
+        zz = self.in_proj(x)
+        q, k, v, g, a = zz[:, : 2 * H * (d + dv) + sp.decay_rank].split([H * d, H * d, H * dv, H * dv, sp.decay_rank], dim=-1)
+        w = self.decay_up.weight.t()
+        z = torch.mm(a, w, out_dtype=torch.float32) if x.is_cuda and x.dtype != torch.float32 else a.float() @ w.float()
+        bias = self._aux("decay_bias", x.device, lambda: self.decay_bias.detach().float())
+        o = mops.state_scan_gla(q, k, v, z, bias, sp.tau, self._state(kv_cache)["S"], kv_cache.ragged, H, d, dv)
+        o = mops.gated_group_rms_norm(o, self.norm_weight, g, dv, self.cfg.norm_eps, x.dtype, gate_act="silu")
+        return self.o_proj(o)
+
+
 class MixerPair(nn.Module):
     """Mixers side by side: every part reads the same input, its output is RMS-normed over the model width with a plain
     weight of its own, and the results are averaged (in fp32: the sum goes straight into the residual stream).  The paged
-    part uses the layer's pages, the recurrent part the layer's state slot."""
+    part uses the layer's pages, the recurrent parts the layer's state slot."""
 
     def __init__(self, cfg: ModelConfig, spec: MixerSpec, layer_idx: int) -> None:
         super().__init__()
         self.cfg, self.spec, self.layer_idx = cfg, spec, layer_idx
         self.shard_config = None
         self.parts = nn.ModuleList([_build(cfg, p, layer_idx) for p in spec.parts])
+        for (tag, _), m in zip(spec.recurrent_parts, [m for m in self.parts if m.spec.recurrent]):
+            m.state_tag = tag
         self.out_norm_weights = nn.ParameterList([nn.Parameter(torch.ones(cfg.hidden_size)) for _ in spec.parts])
 
     def forward(self, x: torch.Tensor, meta, rope=None, kv_cache=None) -> torch.Tensor:
@@ -456,7 +519,7 @@ class MixerPair(nn.Module):
 
 _KINDS = {"attention": BiasSinkAttention, "lightning": LightningAttention, "channel_delta": ChannelDeltaMixer,
           "latent": LatentAttention, "retention": Retention, "mlstm": MatrixLSTM, "ssd": SelectiveStateSpace,
-          "rglru": GatedLinearRecurrence, "pair": MixerPair, "delta": DeltaMixer}
+          "rglru": GatedLinearRecurrence, "pair": MixerPair, "delta": DeltaMixer, "gla": GatedLinearAttention}
 
 
 def _build(cfg: ModelConfig, spec: MixerSpec, layer_idx: int) -> nn.Module:

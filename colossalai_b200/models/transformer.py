@@ -336,13 +336,15 @@ class MLAttention(nn.Module):
 
 
 class MLP(nn.Module):
-    """Dense feed-forward.  `act` overrides the config's activation for this layer; "polynorm" is the non-gated unit
+    """Dense feed-forward.  `act` overrides the config's activation for this layer; "clamped" is the gated unit
+    W_down (g sigmoid(1.702 g) (u + 1)) with g = min(W_gate h, limit), u = clamp(W_up h, -limit, limit); "polynorm" is the non-gated unit
     W_down (a N(z) + b N(z^2) + c N(z^3) + e) with z = W_up h, powers taken element by element, N the division of a token's
     vector by its root mean square, and (a, b, c, e) = `act_coef` learned per layer."""
 
-    def __init__(self, cfg: ModelConfig, intermediate_size: Optional[int] = None, act: Optional[str] = None) -> None:
+    def __init__(self, cfg: ModelConfig, intermediate_size: Optional[int] = None, act: Optional[str] = None,
+                 limit: float = 7.0) -> None:
         super().__init__()
-        self.cfg = cfg
+        self.cfg, self.limit = cfg, limit
         inter = intermediate_size or cfg.intermediate_size
         self.intermediate_size = inter
         self.act = act or cfg.hidden_act
@@ -350,7 +352,7 @@ class MLP(nn.Module):
             self.up_proj = nn.Linear(cfg.hidden_size, inter, bias=False)
             self.act_coef = nn.Parameter(torch.tensor([1.0, 0.0, 0.0, 0.0]))
             self._coef32: Dict[str, torch.Tensor] = {}
-        elif cfg.glu:
+        elif cfg.glu or self.act == "clamped":
             self.gate_up_proj = nn.Linear(cfg.hidden_size, 2 * inter, bias=cfg.mlp_bias)
         else:
             self.up_proj = nn.Linear(cfg.hidden_size, inter, bias=cfg.mlp_bias)
@@ -368,6 +370,8 @@ class MLP(nn.Module):
             if key not in self._coef32:                   # the four numbers in fp32 on the device, built once
                 self._coef32[key] = self.act_coef.detach().float().contiguous()
             h = ops.mixers.poly_norm(self.up_proj(x), self._coef32[key], self.cfg.norm_eps)
+        elif self.act == "clamped":
+            h = ops.clamped_glu(self.gate_up_proj(x), self.limit)
         elif self.cfg.glu:
             h = ops.glu(self.gate_up_proj(x), self.cfg.hidden_act)
         else:
@@ -409,7 +413,7 @@ class DecoderLayer(nn.Module):
 
             self.mlp = RoutedExpertFF(cfg, spec.moe)
         elif spec is not None:
-            self.mlp = MLP(cfg, spec.ff, act=spec.ff_act) if spec.ff is not None else None
+            self.mlp = MLP(cfg, spec.ff, act=spec.ff_act, limit=spec.ff_limit) if spec.ff is not None else None
         elif moe is not None and layer_idx >= moe.first_k_dense_replace and (layer_idx % moe.moe_layer_freq == 0):
             from .moe import SparseMoE
 

@@ -1,11 +1,12 @@
 """Python face of the sequence-mixer kernels (kernel/csrc/mixers.cu): short causal convolution with a carried window,
 recurrent state scans (decayed outer-product state with optional rotary positions, gated delta rule, per-token gated
-outer-product state for selective state spaces and the exponentially gated matrix memory, per-channel gated linear
-recurrence), group RMS norm with a sigmoid / silu gate before or after the norm, rotary positions + unit norm of q / k
+outer-product state for selective state spaces and the exponentially gated matrix memory, outer-product state with a decay
+per key channel, per-channel gated linear recurrence), group RMS norm with a sigmoid / silu gate before or after the norm, rotary positions + unit norm of q / k
 heads, the mean of RMS-normed mixer outputs, RMS norm of a sublayer's output added to an fp32 residual stream, sums into the fp32 stream
 fused with the next RMS / layer norm or with elementwise tanh norms on both sides of the sum, rotary positions from an
-fp32 angle table (alone, or in one pass with the write of the key / value pages), the cache rows of latent attention, and
-paged attention with a distance-bucket bias and a softmax sink (values optionally read from the key rows).
+fp32 angle table (alone, or in one pass with the write of the key / value pages, or with a short convolution in front and a
+unit norm behind it), the cache rows of latent attention, and paged attention with a distance-bucket bias, soft-capped scores,
+a softmax sink and a gate per head (values optionally read from the key rows).
 
 All ops take a RAGGED step (`RaggedMeta`): for every live sequence its next tokens, how many tokens earlier steps
 consumed, and the slot that holds its carried state.  CUDA tensors go to the sm_100a kernels; CPU tensors take the plain
@@ -29,7 +30,8 @@ __all__ = ["RaggedMeta", "short_conv_silu", "state_scan_decay", "state_scan_delt
            "rms_norm_residual", "rms_norm_f32in", "paged_kv_write_mix", "paged_bias_attention", "log_bucket_starts",
            "bucket_lut", "rotary_table", "rotary_half", "stream_add_norm", "latent_kv_write", "state_scan_ssd",
            "state_scan_mlstm", "lru_scan", "rotary_unit_norm", "sigmoid_gate_mul", "norm_mean", "depth_mix", "poly_norm",
-           "head_rms_norm", "distance_slopes", "stream_tanh_norm", "rotary_kv_write"]
+           "head_rms_norm", "distance_slopes", "stream_tanh_norm", "rotary_kv_write", "conv_rotary_kv_write",
+           "state_scan_gla"]
 
 _lib = None
 _SPLIT_BELOW_TILES = 148        # attention steps with fewer CTAs than SMs split their keys
@@ -165,12 +167,22 @@ def rotary_frequencies(dims: int, base: float, scaling: Optional[Sequence[float]
     the slow frequencies for contexts beyond the n positions the model was trained on: with
     d(t) = dims ln(n / (2 pi t)) / (2 ln base) - the channel that turns t times over n positions - lo = max(floor(d(fast)), 0),
     hi = min(ceil(d(slow)), dims - 1) and r_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1), the frequency becomes
-    f_i / s * r_i + f_i * (1 - r_i), and cos and sin are multiplied by 0.1 ln(s) + 1."""
+    f_i / s * r_i + f_i * (1 - r_i), and cos and sin are multiplied by 0.1 ln(s) + 1.  `scaling` = ("wavelength", s, low,
+    high, n) goes by the wavelength 2 pi / f_i: with m_i = clamp((n / wavelength - low) / (high - low), 0, 1) the frequency
+    becomes (1 - m_i) f_i / s + m_i f_i (waves shorter than n / high stay, those longer than n / low are divided by s)."""
     f = torch.tensor(float(base), dtype=torch.float64) ** (-torch.arange(0, dims, 2, dtype=torch.float64) / dims)
     if not scaling:
         return f, 1.0
     if len(scaling) == 1:
         return f / float(scaling[0]), 1.0
+    if scaling[0] == "wavelength":
+        s, low, high, n = [float(v) for v in scaling[1:]]
+        turns = n * f / (2.0 * math.pi)                                            # n / wavelength
+        if high > low:
+            m = ((turns - low) / (high - low)).clamp(0.0, 1.0)
+        else:
+            m = (turns >= low).double()
+        return (1.0 - m) * f / s + m * f, 1.0
     s, n, fast, slow = [float(v) for v in scaling]
     d = lambda t: dims * math.log(n / (2.0 * math.pi * t)) / (2.0 * math.log(base))
     lo = max(math.floor(d(fast)), 0)
@@ -184,7 +196,8 @@ def rotary_table(min_len: int, dims: int, base: float, device, scaling: Optional
     `rotary_frequencies(dims, base, scaling)`.  Angles are formed in float64 and rounded once.  The table is cached per
     (dims, base, scaling, device) and grows in powers of two, so that positions far beyond any configured length stay
     exact."""
-    key = (int(dims), float(base), tuple(float(v) for v in scaling) if scaling else None, str(device))
+    key = (int(dims), float(base), tuple(v if isinstance(v, str) else float(v) for v in scaling) if scaling else None,
+           str(device))
     tab = _rotary_tables.get(key)
     if tab is None or tab.shape[0] < min_len:
         n = max(1024, 1 << max(int(min_len) - 1, 1).bit_length())
@@ -200,33 +213,37 @@ def distance_slopes(heads: int) -> torch.Tensor:
     return torch.tensor([2.0 ** (-8.0 * (h + 1) / heads) for h in range(heads)], dtype=torch.float64).float()
 
 
-def _rot_ref(x: torch.Tensor, pos: torch.Tensor, table: torch.Tensor, dims: int) -> torch.Tensor:
-    """x [T, H, w] fp32: channel i < dims / 2 of every head is paired with channel i + dims / 2."""
+def _rot_ref(x: torch.Tensor, pos: torch.Tensor, table: torch.Tensor, dims: int, interleaved: bool = False) -> torch.Tensor:
+    """x [T, H, w] fp32: channel i < dims / 2 of every head is paired with channel i + dims / 2 (2i with 2i + 1)."""
     half = dims // 2
     cs = table[pos.long()]
     c, sn = cs[:, None, :half], cs[:, None, half:]
+    if interleaved:
+        u, v = x[..., 0:dims:2], x[..., 1:dims:2]
+        rot = torch.stack([u * c - v * sn, v * c + u * sn], -1).reshape(x.shape[:-1] + (dims,))
+        return torch.cat([rot, x[..., dims:]], -1)
     u, v = x[..., :half], x[..., half:dims]
     return torch.cat([u * c - v * sn, v * c + u * sn, x[..., dims:]], -1)
 
 
 def rotary_half(src: torch.Tensor, dst: torch.Tensor, heads: int, src_head_stride: int, src_off: int,
                 dst_head_stride: int, dst_off: int, width: int, dims: int, table: torch.Tensor,
-                token_pos: torch.Tensor) -> None:
+                token_pos: torch.Tensor, interleaved: bool = False) -> None:
     """For every token t and head h: dst[t, h * dst_head_stride + dst_off + (0..width)] = the `width` channels at
     src[t, h * src_head_stride + src_off + ..] with the first `dims` of them turned by the token's position (rotate-half
-    pairs, fp32 arithmetic, one rounding into dst's dtype)."""
+    pairs, with `interleaved` pairs of neighbours; fp32 arithmetic, one rounding into dst's dtype)."""
     T = src.shape[0]
     if use_native(src):
         assert src.stride(1) == 1 and dst.stride(1) == 1 and table.dtype == torch.float32 and table.shape[1] == dims
         loader.check(_get_lib().cb_rotary_half(
             loader.ptr(src), _i64(src.stride(0)), loader.ptr(dst), _i64(dst.stride(0)), _i64(T), heads, src_head_stride,
-            src_off, dst_head_stride, dst_off, width, dims, loader.ptr(table), loader.ptr(token_pos), code(src.dtype),
-            code(dst.dtype), loader.stream_ptr()), "rotary_half")
+            src_off, dst_head_stride, dst_off, width, dims, int(interleaved), loader.ptr(table), loader.ptr(token_pos),
+            code(src.dtype), code(dst.dtype), loader.stream_ptr()), "rotary_half")
         loader.launch_counter.add("rotary_half")
         return
     cols = (torch.arange(heads)[:, None] * src_head_stride + src_off + torch.arange(width)[None, :]).reshape(-1)
     x = src[:, cols].float().view(T, heads, width)
-    y = _rot_ref(x, token_pos, table, dims)
+    y = _rot_ref(x, token_pos, table, dims, interleaved)
     dcols = (torch.arange(heads)[:, None] * dst_head_stride + dst_off + torch.arange(width)[None, :]).reshape(-1)
     dst[:, dcols] = y.reshape(T, heads * width).to(dst.dtype)
 
@@ -271,7 +288,7 @@ def short_conv_silu(x: torch.Tensor, weight: torch.Tensor, state: torch.Tensor, 
 # ------------------------------------------------------------------------------------------------ state scans
 def _scan_native(mode, q, k, v, araw, braw, head_decay, a_log, dt_bias, state, meta, heads, qk_heads, dim, vdim,
                  act_silu, unit_qk, unit_eps, q_scale, k_scale=1.0, rot_table=None, rot_dims=0, gate_cap=0.0,
-                 gate_kind=0, state_n=None, state_m=None):
+                 gate_kind=0, state_n=None, state_m=None, tau=1.0):
     T = q.shape[0]
     out = torch.empty(T, heads * vdim, dtype=torch.float32, device=q.device)
     for t in (q, k, v):
@@ -287,7 +304,7 @@ def _scan_native(mode, q, k, v, araw, braw, head_decay, a_log, dt_bias, state, m
         loader.ptr(out), loader.ptr(work), _i64(T), loader.ptr(meta.cu_q), loader.ptr(meta.ctx_len),
         loader.ptr(meta.slots), meta.nseq, heads, qk_heads, dim, vdim, int(act_silu), int(unit_qk), _f(unit_eps),
         _f(q_scale), _f(k_scale), loader.ptr(rot_table), int(rot_dims if rot_table is not None else 0),
-        loader.ptr(meta.token_pos), int(gate_kind), _f(gate_cap), loader.ptr(state_n), loader.ptr(state_m),
+        loader.ptr(meta.token_pos), int(gate_kind), _f(gate_cap), loader.ptr(state_n), loader.ptr(state_m), _f(tau),
         code(q.dtype), loader.stream_ptr()), "state_scan")
     loader.launch_counter.add("state_scan", 3 if gate_kind == 2 else 2)
     return out
@@ -372,6 +389,39 @@ def state_scan_delta(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay_pr
             u = beta[t][:, None] * (vv[t] - torch.einsum("hdv,hd->hv", S, kk[t]))
             S = S + kk[t][:, :, None] * u[:, None, :]
             out[t0 + t] = torch.einsum("hdv,hd->hv", S, qq[t]).reshape(-1)
+        state[slot] = S
+        t0 += n
+    return out
+
+
+def state_scan_gla(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay_pre: torch.Tensor, decay_bias: torch.Tensor,
+                   tau: float, state: torch.Tensor, meta: RaggedMeta, heads: int, dim: int, vdim: int,
+                   q_scale: Optional[float] = None) -> torch.Tensor:
+    """Gated linear attention.  Per token and head: row decays r = sigmoid(decay_pre + decay_bias)^(1 / tau); the head's matrix
+    M [dim, vdim] becomes diag(r) M + outer(k, v) and is read after the write, y = M^T q (q times `q_scale`, default dim^-1/2).
+    q, k [T, heads x dim], v [T, heads x vdim]; decay_pre [T, heads x dim] fp32, decay_bias [heads x dim] fp32; state [slots,
+    heads, dim, vdim] fp32.  Returns fp32 y [T, heads x vdim]."""
+    if dim > 256:
+        raise NotImplementedError("state_scan: key width above 256 is not supported")
+    q_scale = dim ** -0.5 if q_scale is None else q_scale
+    assert decay_pre.dtype == torch.float32 and decay_bias.dtype == torch.float32
+    if use_native(q):
+        assert decay_pre.stride(1) == 1
+        return _scan_native(3, q, k, v, decay_pre, None, None, None, decay_bias, state, meta, heads, heads, dim, vdim,
+                            False, False, 0.0, q_scale, tau=tau)
+    T = q.shape[0]
+    out = torch.empty(T, heads * vdim, dtype=torch.float32)
+    r = torch.exp(F.logsigmoid(decay_pre + decay_bias) * (1.0 / tau)).view(T, heads, dim)
+    qq, kk = q.float().reshape(T, heads, dim) * q_scale, k.float().reshape(T, heads, dim)
+    vv = v.float().reshape(T, heads, vdim)
+    t0 = 0
+    for n, c, slot in zip(meta.q_lens, meta.ctx_lens, meta.slot_list):
+        if n == 0:
+            continue
+        S = state[slot].clone() if c > 0 else torch.zeros_like(state[slot])
+        for t in range(t0, t0 + n):
+            S = r[t][:, :, None] * S + kk[t][:, :, None] * vv[t][:, None, :]
+            out[t] = torch.einsum("hdv,hd->hv", S, qq[t]).reshape(-1)
         state[slot] = S
         t0 += n
     return out
@@ -738,16 +788,7 @@ def rotary_unit_norm(x: torch.Tensor, heads: int, dim: int, rot_dims: int, inter
         return
     y = x[:, : heads * dim].float().reshape(T, heads, dim)
     if rot_dims:
-        half = rot_dims // 2
-        cs = table[token_pos.long()]
-        c, sn = cs[:, None, :half], cs[:, None, half:]
-        if interleaved:
-            a, b = y[..., 0:rot_dims:2], y[..., 1:rot_dims:2]
-            rot = torch.stack([a * c - b * sn, b * c + a * sn], -1).reshape(T, heads, rot_dims)
-        else:
-            a, b = y[..., :half], y[..., half:rot_dims]
-            rot = torch.cat([a * c - b * sn, b * c + a * sn], -1)
-        y = torch.cat([rot, y[..., rot_dims:]], -1)
+        y = _rot_ref(y, token_pos, table, rot_dims, interleaved)
     if unit_eps is not None:
         y = y / torch.sqrt((y * y).mean(-1, keepdim=True) + unit_eps)
     x[:, : heads * dim] = y.reshape(T, heads * dim).to(x.dtype)
@@ -777,6 +818,42 @@ def rotary_kv_write(qkv: torch.Tensor, heads: int, kv_heads: int, dim: int, vdim
     rotary_unit_norm(qkv, heads + kv_heads, dim, rot_dims, False, table, meta.token_pos, None)
     a, b = heads * dim, (heads + kv_heads) * dim
     paged_kv_write_mix(qkv[:, a:b], qkv[:, b:b + kv_heads * vdim], k_cache, v_cache, block_tables, meta)
+
+
+def conv_rotary_kv_write(x: torch.Tensor, weight: torch.Tensor, state: torch.Tensor, heads: int, kv_heads: int, dim: int,
+                         vdim: int, rot_dims: int, interleaved: bool, table: Optional[torch.Tensor],
+                         unit_eps: Optional[float], k_cache: torch.Tensor, v_cache: torch.Tensor,
+                         block_tables: torch.Tensor, meta: RaggedMeta) -> torch.Tensor:
+    """One pass over projection rows q | k | v [T, heads x dim + kv_heads x (dim + vdim)] (unit stride inside a row): the short
+    causal convolution of `short_conv_silu` on every channel (no activation, no bias; `weight` [C, taps], `state` [slots,
+    taps - 1, C] read and advanced), then on the q and k heads rotary positions and the unit norm of `rotary_unit_norm`, all in
+    fp32 with one rounding at the end.  Queries are returned [T, heads x dim]; keys and values go into the tokens' rows of
+    `k_cache` [blocks, block_size, kv_heads, dim] / `v_cache` [.., kv_heads, vdim]."""
+    T, C = x.shape
+    taps = weight.shape[1]
+    bs = k_cache.shape[1]
+    a, b = heads * dim, (heads + kv_heads) * dim
+    assert C == b + kv_heads * vdim and weight.shape[0] == C
+    assert k_cache.shape[2:] == (kv_heads, dim) and v_cache.shape[2:] == (kv_heads, vdim)
+    vec = dim % 4 == 0 and vdim % 4 == 0 and x.stride(0) % 4 == 0 and x.data_ptr() % (4 * x.element_size()) == 0
+    if use_native(x) and taps <= 4 and max(dim, vdim) <= (256 if vec else 128):
+        assert x.stride(1) == 1 and weight.is_contiguous() and weight.dtype == x.dtype
+        assert state.is_contiguous() and state.dtype == x.dtype
+        assert k_cache.dtype == x.dtype and v_cache.dtype == x.dtype and k_cache.is_contiguous() and v_cache.is_contiguous()
+        assert rot_dims == 0 or (table.dtype == torch.float32 and table.shape[1] == rot_dims)
+        q = torch.empty(T, a, dtype=x.dtype, device=x.device)
+        loader.check(_get_lib().cb_conv_rotary_kv_write(
+            loader.ptr(x), _i64(x.stride(0)), loader.ptr(weight), loader.ptr(state), taps, loader.ptr(q), heads, kv_heads, dim,
+            vdim, rot_dims, int(interleaved), loader.ptr(table if rot_dims else None), int(unit_eps is not None),
+            _f(unit_eps or 0.0), loader.ptr(k_cache), loader.ptr(v_cache), loader.ptr(block_tables), loader.ptr(meta.cu_q),
+            loader.ptr(meta.ctx_len), loader.ptr(meta.slots), meta.nseq, meta.max_q, bs, block_tables.shape[1], int(vec),
+            code(x.dtype), loader.stream_ptr()), "conv_rotary_kv_write")
+        loader.launch_counter.add("conv_rotary_kv_write", 2 if taps > 1 else 1)
+        return q
+    y = short_conv_silu(x, weight, state, meta, activation=False)       # (also more taps / wider heads on the GPU)
+    rotary_unit_norm(y, heads + kv_heads, dim, rot_dims, interleaved, table, meta.token_pos, unit_eps)
+    paged_kv_write_mix(y[:, a:b], y[:, b:], k_cache, v_cache, block_tables, meta)
+    return y[:, :a].contiguous()
 
 
 _NORM_KINDS = {None: 0, "none": 0, "rms": 1, "layer": 2}
@@ -865,9 +942,10 @@ def stream_tanh_norm(x: torch.Tensor, y: Optional[torch.Tensor] = None, out_norm
 
 # ------------------------------------------------------------------------------------------------ paged attention
 def latent_kv_write(z: torch.Tensor, norm_weight: torch.Tensor, eps: float, kv_rank: int, rot_table: torch.Tensor,
-                    cache: torch.Tensor, block_tables: torch.Tensor, meta: RaggedMeta) -> None:
+                    cache: torch.Tensor, block_tables: torch.Tensor, meta: RaggedMeta, interleaved: bool = False) -> None:
     """The cache rows of latent attention.  z [T, kv_rank + rot]: the first `kv_rank` columns are RMS-normalised with
-    `norm_weight` (the latent), the others are turned by the token's position (the rotated key part all heads share);
+    `norm_weight` (the latent), the others are turned by the token's position (the rotated key part all heads share;
+    rotate-half pairs, or neighbours with `interleaved`);
     both go, rounded once, into the token's row of the paged cache [blocks, block_size, 1, kv_rank + rot]."""
     T, Wz = z.shape
     rot = Wz - kv_rank
@@ -876,7 +954,7 @@ def latent_kv_write(z: torch.Tensor, norm_weight: torch.Tensor, eps: float, kv_r
         assert z.stride(1) == 1 and cache.is_contiguous() and cache.shape[-1] == Wz and rot_table.shape[1] == rot
         loader.check(_get_lib().cb_latent_kv_write(
             loader.ptr(z), _i64(z.stride(0)), loader.ptr(norm_weight), code(norm_weight.dtype), _f(eps), kv_rank, rot,
-            loader.ptr(rot_table), loader.ptr(cache), loader.ptr(block_tables), loader.ptr(meta.token_seq),
+            int(interleaved), loader.ptr(rot_table), loader.ptr(cache), loader.ptr(block_tables), loader.ptr(meta.token_seq),
             loader.ptr(meta.token_pos), _i64(T), bs, block_tables.shape[1], code(z.dtype), loader.stream_ptr()),
             "latent_kv_write")
         loader.launch_counter.add("latent_kv_write")
@@ -884,7 +962,7 @@ def latent_kv_write(z: torch.Tensor, norm_weight: torch.Tensor, eps: float, kv_r
     zf = z.float()
     c = zf[:, :kv_rank]
     c = c / torch.sqrt((c * c).mean(-1, keepdim=True) + eps) * norm_weight.float()
-    kr = _rot_ref(zf[:, None, kv_rank:], meta.token_pos, rot_table, rot)[:, 0]
+    kr = _rot_ref(zf[:, None, kv_rank:], meta.token_pos, rot_table, rot, interleaved)[:, 0]
     blk = block_tables[meta.token_seq.long(), (meta.token_pos // bs).long()].long()
     off = (meta.token_pos % bs).long()
     cache.view(cache.shape[0], bs, Wz)[blk, off] = torch.cat([c, kr], -1).to(cache.dtype)
@@ -931,7 +1009,8 @@ def paged_bias_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.
                          lut: Optional[torch.Tensor] = None, tensor_cores: Optional[bool] = None,
                          vdim: Optional[int] = None, mask_block: int = 0, wide_weights: bool = False,
                          sink_values: Optional[torch.Tensor] = None, slopes: Optional[torch.Tensor] = None,
-                         window: int = 0, keep_first: int = 0) -> torch.Tensor:
+                         window: int = 0, keep_first: int = 0, softcap: float = 0.0,
+                         head_gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal attention of every step token over positions 0..pos of its sequence in the paged cache; with `mask_block`
     only over the positions of its own block, floor(pos / mask_block) * mask_block .. pos (blocks are counted from the
     start of the sequence, whatever the step's cut).
@@ -942,7 +1021,9 @@ def paged_bias_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.
     score 0 without a value to the softmax - with `sink_values` [heads] fp32 a key of that (unscaled) score per head.
     `slopes` [heads] fp32 takes slope * (pos - key position) off every score; `window` > 0 keeps only the keys
     pos - window + 1 .. pos and the first `keep_first` keys of the sequence (at their true positions, whatever the window or
-    block mask says).  Returns [T, heads x vdim].
+    block mask says).  `softcap` > 0 passes scale * q.k through softcap * tanh(. / softcap) before bias and slope (the sink
+    stays as it is).  `head_gate` [T, heads] (unit stride inside a row): every head's output times sigmoid of its gate.
+    Returns [T, heads x vdim].
 
     Two kernels: 16-bit inputs whose head widths are multiples of 8 up to 256 run on tensor cores (`lut` = `bucket_lut`
     of the same buckets; built here when absent); everything else - fp32 above all - takes the exact CUDA-core kernel.
@@ -959,6 +1040,8 @@ def paged_bias_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.
         if vdim > 512:
             raise NotImplementedError("paged_bias_attention: value width above 512 is not supported")
         assert q.stride(1) == 1 and k_cache.dtype == q.dtype and v_cache.dtype == q.dtype
+        assert head_gate is None or (head_gate.shape == (T, heads) and head_gate.stride(1) == 1 and head_gate.dtype == q.dtype)
+        gargs = (loader.ptr(head_gate), _i64(0 if head_gate is None else head_gate.stride(0)))
         out = torch.empty(T, heads * vdim, dtype=q.dtype, device=q.device)
         mma_ok = (q.dtype in (torch.bfloat16, torch.float16) and dim % 8 == 0 and vdim % 8 == 0 and dim <= 256
                   and vdim <= 256 and nb <= 255 and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0 and ldv % 8 == 0)
@@ -990,7 +1073,7 @@ def paged_bias_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.
                 loader.ptr(bias_table), loader.ptr(lut), 0 if lut is None else lut.numel(), nb, loader.ptr(out), _i64(T), meta.nseq, meta.max_q,
                 heads, G, dim, vdim, ldv, bs, block_tables.shape[1], _f(scale), int(sink), chunk, splits,
                 loader.ptr(part_o), loader.ptr(part_ml), int(mask_block), int(wide_weights), loader.ptr(sink_values),
-                loader.ptr(slopes), int(window), int(keep_first), code(q.dtype), loader.stream_ptr()),
+                loader.ptr(slopes), int(window), int(keep_first), _f(softcap), *gargs, code(q.dtype), loader.stream_ptr()),
                 "paged_bias_attention_mma")
             loader.launch_counter.add("paged_bias_attention_mma")
             return out
@@ -998,8 +1081,8 @@ def paged_bias_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.
             loader.ptr(q), _i64(q.stride(0)), loader.ptr(k_cache), loader.ptr(v_cache), loader.ptr(block_tables),
             loader.ptr(meta.token_seq), loader.ptr(meta.token_pos), loader.ptr(bias_table), loader.ptr(bucket_starts), nb,
             loader.ptr(out), _i64(T), heads, G, dim, vdim, ldv, bs, block_tables.shape[1], _f(scale), int(sink),
-            int(mask_block), loader.ptr(sink_values), loader.ptr(slopes), int(window), int(keep_first), code(q.dtype),
-            loader.stream_ptr()), "paged_bias_attention")
+            int(mask_block), loader.ptr(sink_values), loader.ptr(slopes), int(window), int(keep_first), _f(softcap), *gargs,
+            code(q.dtype), loader.stream_ptr()), "paged_bias_attention")
         loader.launch_counter.add("paged_bias_attention")
         return out
     out = torch.empty(T, heads * vdim, dtype=q.dtype)
@@ -1014,6 +1097,8 @@ def paged_bias_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.
         vv = v_cache[blks].reshape(-1, G, ldv)[:L, :, :vdim].float().repeat_interleave(rep, 1)
         qq = q[t0:t0 + n].float().view(n, heads, dim)
         s = torch.einsum("ihd,jhd->hij", qq, kk) * scale
+        if softcap:
+            s = softcap * torch.tanh(s / softcap)
         dist = torch.arange(c, L)[:, None] - torch.arange(L)[None, :]
         if bias_table is not None:
             b = torch.bucketize(dist.clamp(min=0), bucket_starts.to(torch.int64), right=True) - 1
@@ -1031,6 +1116,9 @@ def paged_bias_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.
             sv = torch.zeros(heads) if sink_values is None else sink_values.float()
             s = torch.cat([s, sv[:, None, None].expand(heads, n, 1)], -1)
         p = torch.softmax(s, -1)[..., :L]
-        out[t0:t0 + n] = torch.einsum("hij,jhv->ihv", p, vv).reshape(n, heads * vdim).to(q.dtype)
+        o = torch.einsum("hij,jhv->ihv", p, vv)
+        if head_gate is not None:
+            o = o * torch.sigmoid(head_gate[t0:t0 + n].float())[:, :, None]
+        out[t0:t0 + n] = o.reshape(n, heads * vdim).to(q.dtype)
         t0 += n
     return out
