@@ -8,9 +8,12 @@ for the Pogorax family (pairs of attention and a recurrent mixer side by side, s
 delta rule with a decay per head, grouped output norms, a depth-weighted stream, normalised-power and routed feed-forwards).
 `--family sodurax` runs the Sodurax family (windowed attention that keeps the first keys, tanh norms on both sides of every
 sublayer, sigmoid-routed squared-ReLU experts, layers that run twice) beside Domorax, the closest served family.
+`--family sumolorn` runs the Sumolorn family (soft-capped windowed attention with sinks and head gates, latent attention, pairs
+of convolved attention and gated linear attention, clamped gated feed-forwards, layers that run twice) beside Pogorax, the
+other family of pairs on a pre-norm fp32 stream.
 
     python examples/inference/benchmark_hybrid.py [--sizes 2048x8,4096x4] [--batch 8] [--in_len 2048] [--out_len 64]
-                                                  [--family gopunex|palilix|pogorax|domorax|sodurax]
+                                                  [--family gopunex|palilix|pogorax|domorax|sodurax|sumolorn]
 
 Also reachable as `python bench.py --workload hybrid-serve`.  One JSON line per (size, family) and one per kernel.
 Timing: CUDA events on the launching stream after warm-up; the kernel timings write a 256 MB buffer between runs (L2
@@ -141,6 +144,33 @@ def sodurax_config(width: int, layers: int, vocab: int = 32000) -> ModelConfig:
                        tie_word_embeddings=True, max_position_embeddings=1 << 20)
 
 
+def sumolorn_config(width: int, runs: int, vocab: int = 32000, kv_rank: int = 192, rot: int = 64) -> ModelConfig:
+    """`runs` layer runs [latent, pair, capped attention, latent, ...] of which a span from the second layer on (two layers,
+    one in short models) runs twice.  Heads of 128 channels, one key head per four query heads, the first 64 channels rotated;
+    windows of 1024 positions, a cap of 50; latent rows of kv_rank + rot = 256 columns behind a query latent of 3/8 of the
+    width; gated linear attention with heads of 64 x 128; gated feed-forwards of 8/3 x width clamped at 7."""
+    H, d = width // 128, 128
+    G = max(H // 4, 1)
+    att = MixerSpec(kind="attention", heads=H, kv_heads=G, dim=d, vdim=d, scale=d ** -0.5, rot_dims=64, rot_base=5e5,
+                    rot_scaling=["wavelength", 4.0, 1.0, 4.0, 4096.0], window=1024, softcap=50.0, sink_learned=True,
+                    head_gate=True, wide_weights=True)
+    lat = MixerSpec(kind="latent", heads=H, kv_heads=1, dim=d - rot, rot_dim=rot, rot_dims=rot, vdim=d, kv_rank=kv_rank,
+                    rot_base=5e5, rot_interleaved=True, scale=d ** -0.5, q_rank=width * 3 // 8, sink_learned=True,
+                    head_gate=True, wide_weights=True)
+    left = MixerSpec(kind="attention", heads=H, kv_heads=G, dim=d, vdim=d, scale=d ** -0.5, rot_dims=64, rot_base=5e5, conv=4,
+                     conv_values=True, head_unit_norm=True, window=1024, wide_weights=True)
+    right = MixerSpec(kind="gla", heads=H, dim=64, vdim=d, tau=16.0, decay_rank=16)
+    ff = width * 8 // 3 // 64 * 64
+    order = [lat, MixerSpec(kind="pair", parts=[left, right]), att]
+    span = 2 if runs >= 6 else 1
+    own = runs - span
+    specs = [LayerSpec(mixer=order[i % 3], ff=ff, ff_act="clamped", ff_limit=7.0) for i in range(own)]
+    return ModelConfig(model_type="sumolorn", vocab_size=vocab, hidden_size=width, intermediate_size=ff, layer_specs=specs,
+                       layer_order=[0] + list(range(1, 1 + span)) * 2 + list(range(1 + span, own)), norm_eps=1e-6,
+                       norm_type="rms", norm_weight_offset=1.0, hidden_act="clamped", glu=True, pos_type="none",
+                       fp32_residual=True, fp32_logits=True, logit_scale=0.25, max_position_embeddings=1 << 20)
+
+
 def llama_config(width: int, layers: int, vocab: int = 32000) -> ModelConfig:
     H = width // 128
     # 8/3 x width gated feed-forward = the parameter count of the hybrid's 4 x width plain one
@@ -157,7 +187,7 @@ def build(cfg: ModelConfig):
         for n, p in model.named_parameters():          # recurrent layers: non-degenerate convolutions and decays
             if n.endswith("conv_weight"):
                 p.normal_(0, 0.5)
-            elif n.endswith("dt_bias") or n.endswith("rel_bias"):
+            elif n.endswith("dt_bias") or n.endswith("rel_bias") or n.endswith("decay_bias"):
                 p.normal_(0, 1.0)
             elif n.endswith("v_mix"):
                 p.fill_(0.4)
@@ -791,6 +821,112 @@ def kernels_sodurax(width: int, batch: int, in_len: int) -> list:
     return rows
 
 
+def kernels_sumolorn(width: int, batch: int, in_len: int, kv_rank: int = 192, rot: int = 64) -> list:
+    """Every kernel of the Sumolorn layers alone at one layer's sizes beside its like kernel of the closest families."""
+    from colossalai_b200 import ops
+    from colossalai_b200.ops import mixers as M
+
+    hbm, tflops, src = peaks()
+    dev, dt = "cuda", torch.bfloat16
+    H, d, bs = width // 128, 128, 64
+    G, ff = max(H // 4, 1), width * 8 // 3 // 64 * 64
+    flush = torch.zeros(64 << 20, dtype=torch.float32, device=dev)
+    rows = []
+
+    def rec(name, phase, ms, bytes_, flops, like=""):
+        ideal = max(bytes_ / hbm, flops / tflops) * 1e3
+        rows.append({"kernel": name, "phase": phase + ("(graph replay)" if phase == "decode" else ""), "width": width,
+                     "ms": ms, "roofline_ms": ideal, "frac_of_" + src + "_roofline": ideal / ms,
+                     "bound": "hbm" if bytes_ / hbm > flops / tflops else "tensor", "like": like})
+
+    for phase, q_len, ctx in (("prefill", in_len, 0), ("decode", 1, in_len)):
+        replay = phase == "decode"             # decode kernels are timed as graph replays (no host share)
+        T = batch * q_len
+        L = ctx + q_len
+        meta = M.RaggedMeta.build([q_len] * batch, [ctx] * batch, list(range(batch)), dev)
+        x = lambda c: torch.randn(T, c, device=dev, dtype=dt)
+        t = lambda fn: _time(fn, flush, graph=replay)
+        per = (L + bs - 1) // bs
+        kc, vc = (torch.randn(batch * per, bs, G, d, device=dev, dtype=dt) for _ in range(2))
+        tables = torch.arange(batch * per, dtype=torch.int32, device=dev).view(batch, per)
+        tab = M.rotary_table(L + 1, 64, 5e5, dev, ["wavelength", 4.0, 1.0, 4.0, 4096.0])
+        # convolution + rotation + unit norm + page write in one pass  |  like: the chain of single kernels (Pogorax rotation +
+        # unit norm behind the convolution of the recurrent families)
+        C = (H + 2 * G) * d
+        qkv, w4, st = x(C), torch.randn(C, 4, device=dev, dtype=dt), torch.zeros(batch, 3, C, device=dev, dtype=dt)
+        rec("conv_rotary_kv_write(4 taps, 64 of 128, unit norm)", phase,
+            t(lambda: M.conv_rotary_kv_write(qkv, w4, st, H, G, d, d, 64, False, tab, 1e-6, kc, vc, tables, meta)),
+            2 * T * C * 2, 0, like="short_conv_silu / rotary_unit_norm / paged_kv_write_mix")
+        rec("gopunex:short_conv_silu", phase, t(lambda: M.short_conv_silu(qkv, w4, st, meta)), 2 * T * C * 2, 0)
+        rec("pogorax:rotary_unit_norm", phase,
+            t(lambda: M.rotary_unit_norm(qkv, H + G, d, 64, True, tab, meta.token_pos, 1e-6)), 2 * T * (H + G) * d * 2, 0)
+        kk, vv = qkv[:, H * d:(H + G) * d], qkv[:, (H + G) * d:]
+        rec("gopunex:paged_kv_write_mix", phase, t(lambda: M.paged_kv_write_mix(kk, vv, kc, vc, tables, meta)),
+            2 * T * 2 * G * d * 2, 0)
+        rec("rotary_kv_write(64 of 128)", phase, t(lambda: M.rotary_kv_write(qkv, H, G, d, d, 64, tab, kc, vc, tables, meta)),
+            T * (2 * H * 64 + 4 * G * d) * 2, 0, like="(sodurax: same kernel)")
+        # attention inside a window of 1024: soft cap + sinks + head gates; without them  |  like: Sodurax window attention
+        qa, gate, sinks = x(H * d), x(H + 8)[:, :H], torch.randn(H, device=dev)
+        win, io = 1024, 2 * T * H * d * 2
+        seen = sum(min(p_ + 1, win) for p_ in range(ctx, L)) * batch
+        wbytes = 2 * batch * min(L, win + q_len) * G * d * 2 + io
+        rec("paged_attention(window 1024, soft cap, sinks, head gates)", phase,
+            t(lambda: M.paged_bias_attention(qa, kc, vc, tables, meta, d ** -0.5, window=win, sink=True, sink_values=sinks,
+                                             softcap=50.0, head_gate=gate, wide_weights=True)), wbytes, 4.0 * H * d * seen,
+            like="paged_attention(window 1024, 4 kept)")
+        rec("paged_attention(window 1024)", phase,
+            t(lambda: M.paged_bias_attention(qa, kc, vc, tables, meta, d ** -0.5, window=win, wide_weights=True)), wbytes,
+            4.0 * H * d * seen, like="paged_attention(window 1024, 4 kept)")
+        rec("sodurax:paged_attention(window 1024, 4 kept)", phase,
+            t(lambda: M.paged_bias_attention(qa, kc, vc, tables, meta, d ** -0.5, window=win, keep_first=4, wide_weights=True)),
+            wbytes, 4.0 * H * d * seen)
+        # latent attention over the whole context: sinks + head gates  |  like: Palilix latent attention
+        W2, every = kv_rank + rot, batch * (q_len * ctx + q_len * (q_len + 1) / 2)
+        lc, qa2 = torch.randn(batch * per, bs, 1, W2, device=dev, dtype=dt), x(H * W2)
+        lb, lf = batch * L * W2 * 2 + T * H * (W2 + kv_rank) * 2, 2.0 * H * (W2 + kv_rank) * every
+        rec("latent_attention(sinks, head gates, two-term weights)", phase,
+            t(lambda: M.paged_bias_attention(qa2, lc, lc, tables, meta, d ** -0.5, vdim=kv_rank, sink=True, sink_values=sinks,
+                                             head_gate=gate, wide_weights=True)), lb, lf, like="latent_attention")
+        rec("palilix:latent_attention", phase,
+            t(lambda: M.paged_bias_attention(qa2, lc, lc, tables, meta, d ** -0.5, vdim=kv_rank)), lb, lf)
+        ltab, wl, zz, qh = M.rotary_table(L + 1, rot, 5e5, dev), torch.ones(kv_rank, device=dev, dtype=dt), x(W2), x(H * d)
+        for name, il in (("latent_kv_write(interleaved)", True), ("palilix:latent_kv_write", False)):
+            rec(name, phase, t(lambda: M.latent_kv_write(zz, wl, 1e-6, kv_rank, ltab, lc, tables, meta, interleaved=il)),
+                2 * T * W2 * 2, 0, like="latent_kv_write" if il else "")
+        for name, il in (("rotary_half(interleaved)", True), ("palilix:rotary_half", False)):
+            rec(name, phase, t(lambda: M.rotary_half(qh, qa2, H, d, d - rot, W2, kv_rank, rot, rot, ltab, meta.token_pos,
+                                                     interleaved=il)), 2 * T * H * rot * 2, 0, like="rotary_half" if il else "")
+        # gated linear attention (heads of 64 x 128)  |  like: the delta rule with channel decays, the decay scan, same sizes
+        dk = 64
+        S = torch.zeros(batch, H, dk, d, device=dev)
+        q, k, v, z = x(H * dk) * 0.1, x(H * dk) * 0.1, x(H * d), torch.randn(T, H * dk, device=dev)
+        zb, a, b = torch.zeros(H * dk, device=dev), x(H * dk), x(H)
+        sb = 2 * S.numel() * 4
+        rec("state_scan_gla", phase, t(lambda: M.state_scan_gla(q, k, v, z, zb, 16.0, S, meta, H, dk, d)),
+            T * (2 * H * dk * 2 + H * dk * 4 + H * d * 2 + H * d * 4) + sb, 4.0 * T * H * dk * d, like="state_scan_delta")
+        al = torch.zeros(H, device=dev)
+        rec("gopunex:state_scan_delta", phase, t(lambda: M.state_scan_delta(q, k, v, a, b, al, zb, S, meta, H, H, dk, d)),
+            T * (3 * H * dk * 2 + H * d * 2 + H * d * 4) + sb, 6.0 * T * H * dk * d)
+        dec = torch.full((H,), 0.97, device=dev)
+        rec("gopunex:state_scan_decay", phase, t(lambda: M.state_scan_decay(q, k, v, dec, S, meta, H, dk, d)),
+            T * (2 * H * dk * 2 + H * d * 2 + H * d * 4) + sb, 4.0 * T * H * dk * d)
+        o, g = torch.randn(T, H * d, device=dev), x(H * d)
+        wn, ww = torch.ones(d, device=dev, dtype=dt), torch.ones(width, device=dev, dtype=dt)
+        rec("gated_group_rmsnorm(silu)", phase, t(lambda: M.gated_group_rms_norm(o, wn, g, d, 1e-6, dt, gate_act="silu")),
+            T * H * d * (4 + 2 + 2), 0, like="(gopunex: same kernel)")
+        # stream, feed-forward
+        xs, y1, y2 = torch.randn(T, width, device=dev), x(width), x(width)
+        rec("stream_add_norm(1 addend, rms)", phase,
+            t(lambda: M.stream_add_norm(xs, [y1], weight=ww, eps=1e-6, kind="rms", offset=1.0)), T * width * (4 + 4 + 2 + 2), 0,
+            like="(pogorax: same kernel)")
+        rec("norm_mean(2 parts)", phase, t(lambda: M.norm_mean([y1, y2], [ww, ww], 1e-6)), T * width * (2 + 2 + 4), 0,
+            like="(pogorax: same kernel)")
+        gu = x(2 * ff)
+        rec("clamped_glu", phase, t(lambda: ops.clamped_glu(gu, 7.0)), 3 * T * ff * 2, 0, like="glu_fwd")
+        rec("pogorax:glu_fwd(gelu_tanh)", phase, t(lambda: ops.glu(gu, "gelu_tanh")), 3 * T * ff * 2, 0)
+    return rows
+
+
 def main(argv=None):
     ap = argparse.ArgumentParser()
     ap.add_argument("--sizes", default="2048x8,4096x4", help="width x layers, comma separated")
@@ -798,9 +934,9 @@ def main(argv=None):
     ap.add_argument("--in_len", type=int, default=2048)
     ap.add_argument("--out_len", type=int, default=32)
     ap.add_argument("--cuda_graph", action="store_true", help="also run both families with CUDA-graph decode steps")
-    ap.add_argument("--family", default="gopunex", choices=["gopunex", "palilix", "pogorax", "domorax", "sodurax"],
+    ap.add_argument("--family", default="gopunex", choices=["gopunex", "palilix", "pogorax", "domorax", "sodurax", "sumolorn"],
                     help="gopunex: the hybrid decoder beside Llama (default).  palilix / pogorax / domorax: that family "
-                         "beside Gopunex, the closest served family; sodurax: beside Domorax")
+                         "beside Gopunex, the closest served family; sodurax: beside Domorax; sumolorn: beside Pogorax")
     ap.add_argument("--no-kernels", action="store_true")
     ap.add_argument("--no-serve", action="store_true")
     args = ap.parse_args(argv)
@@ -813,12 +949,13 @@ def main(argv=None):
                         "palilix": lambda: (palilix_config(width, layers), hybrid_config(width, layers)),
                         "pogorax": lambda: (pogorax_config(width, layers), hybrid_config(width, layers)),
                         "domorax": lambda: (domorax_config(width, layers), hybrid_config(width, layers)),
-                        "sodurax": lambda: (sodurax_config(width, layers), domorax_config(width, layers))}[args.family]()
+                        "sodurax": lambda: (sodurax_config(width, layers), domorax_config(width, layers)),
+                        "sumolorn": lambda: (sumolorn_config(width, layers), pogorax_config(width, layers))}[args.family]()
                 for cfg in pair:
                     print(json.dumps(serve(cfg, args.batch, args.in_len, args.out_len, graph)), flush=True)
         if not args.no_kernels:
             kfn = {"gopunex": kernels, "palilix": kernels_palilix, "pogorax": kernels_pogorax,
-                   "domorax": kernels_domorax, "sodurax": kernels_sodurax}[args.family]
+                   "domorax": kernels_domorax, "sodurax": kernels_sodurax, "sumolorn": kernels_sumolorn}[args.family]
             for row in kfn(width, args.batch, args.in_len):
                 print(json.dumps(row), flush=True)
 

@@ -75,16 +75,15 @@ def causal_conv(x, w):
 
 def weigh(scores, pos, size, sink):
     """scores [L, L] of one head -> softmax weights over the visible keys; a sink score joins the denominator only."""
-    L = scores.shape[0]
-    out = torch.zeros_like(scores)
-    for i in range(L):
-        js = [j for j in range(L) if 0 <= pos[i] - pos[j] and (not size or pos[i] - pos[j] < size)]
-        s = scores[i, js]
-        m = s.max() if sink is None else torch.maximum(s.max(), sink)
-        e = torch.exp(s - m)
-        den = e.sum() + (0.0 if sink is None else torch.exp(sink - m))
-        out[i, js] = e / den
-    return out
+    p = torch.as_tensor(pos)
+    dist = p[:, None] - p[None, :]
+    seen = (dist >= 0) & (dist < size) if size else dist >= 0
+    s = scores.masked_fill(~seen, -math.inf)
+    m = s.max(1, keepdim=True).values
+    if sink is not None:
+        m = torch.maximum(m, sink)
+    e = torch.exp(s - m)
+    return e / (e.sum(1, keepdim=True) + (0.0 if sink is None else torch.exp(sink - m)))
 
 
 # ----------------------------------------------------------------------------------------------- mixers
@@ -302,8 +301,9 @@ def write_checkpoint(folder, cfg, W):
     from safetensors.torch import save_file
 
     os.makedirs(folder, exist_ok=True)
+    plain = dict(cfg, layers=[{k: v for k, v in ly.items() if k != "_rank"} for ly in cfg["layers"]])   # the rank: tensors tell
     with open(os.path.join(folder, "config.json"), "w") as f:
-        json.dump(cfg, f)
+        json.dump(plain, f)
     save_file({k: v.to(torch.bfloat16).contiguous() for k, v in W.items()}, os.path.join(folder, "model.safetensors"))
     return str(folder)
 
