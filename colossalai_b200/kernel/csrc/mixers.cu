@@ -252,11 +252,20 @@ struct ScanParams {
 // Two kernels.  `scan_prepare_kernel` is elementwise and fully parallel: activations, unit norms, decays and write
 // strengths of every token in fp32 into a workspace whose rows are padded to the kernel's key width (q, k: zeros;
 // decay: ones) and value rows to a multiple of SCAN_COLS.  `state_scan_kernel` is the recurrence: a CTA owns SCAN_COLS
-// value columns of one (sequence, head); column j of S lives in the registers of SCAN_PARTS adjacent lanes, each holding
-// DK / SCAN_PARTS of its rows, so S^T k and S^T q are partial sums per lane joined by two shuffles in a fixed order.
+// value columns of one (sequence, head); a lane holds a tile of S, RP rows x SCAN_CPL columns, in registers, so that a value
+// of q, k or the decay that is read from shared memory serves SCAN_CPL columns; PARTS adjacent lanes share the rows of a
+// column group, and S^T k and S^T q are partial sums per lane joined by shuffles in a fixed order.
 // The workspace rows of SCAN_TOK_TILE tokens arrive by cp.async in a two-stage ring while the previous tile is walked.
-constexpr int SCAN_PARTS = 4;
-constexpr int SCAN_COLS = 32;          // 128 threads
+constexpr int SCAN_CPL = 4;            // value columns per lane
+constexpr int SCAN_COLS = 32;          // value columns per CTA
+
+template <int DK> struct ScanTile {
+  static constexpr int PARTS = DK <= 16 ? 4 : DK <= 128 ? 8 : 16;       // lanes that share the rows of a column group
+  static constexpr int RP = DK / PARTS;                                 // rows per lane
+  static constexpr int RPP = RP == 4 ? 4 : RP + 4;                      // a lane's rows in shared memory start this far apart:
+  static constexpr int DKP = PARTS * RPP;                               // the 16-byte reads of 8 lanes hit different banks
+  static constexpr int THREADS = PARTS * SCAN_COLS / SCAN_CPL;
+};
 
 struct ScanWork {
   float *q, *k, *g, *beta, *v;         // [T, qk_heads, DK] x2, [T, heads, DK], [T, heads], [T, heads, VP]
@@ -364,6 +373,47 @@ __global__ void __launch_bounds__(128) scan_prepare_kernel(ScanParams p, ScanWor
   }
 }
 
+template <typename T, int VEC> CB_DEVICE void load_vec(const void* p, bool f32, int64_t i, float (&v)[VEC]);
+
+// The same for rows mode on widths and addresses that allow four channels per access (the launcher checks): nothing there
+// needs more of a row than the channel itself, so a thread takes quads of q, k, decay and value channels as they come.
+template <typename T>
+__global__ void __launch_bounds__(256) scan_prepare_rows_vec_kernel(ScanParams p, ScanWork w) {
+  const int64_t t = blockIdx.x;
+  const int dim = p.dim, dq = w.DK / 4, nq = p.heads * dq, vq = w.VP / 4, items = 3 * nq + p.heads * vq;
+#pragma unroll 4
+  for (int it = threadIdx.x; it < items; it += 256) {
+    float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+    float x[4];
+    if (it < 3 * nq) {
+      const int sec = it < nq ? 0 : (it < 2 * nq ? 1 : 2), r = it - sec * nq, h = r / dq, i = r % dq * 4;
+      if (sec == 2) {
+        o = make_float4(1.f, 1.f, 1.f, 1.f);
+        if (i < dim) {
+          const float4 z = *reinterpret_cast<const float4*>((const float*)p.araw + t * p.lda + h * dim + i);
+          const float4 b = *reinterpret_cast<const float4*>(p.dt_bias + h * dim + i);
+          o.x = expf(logsigmoid_f(z.x + b.x) * p.inv_tau); o.y = expf(logsigmoid_f(z.y + b.y) * p.inv_tau);
+          o.z = expf(logsigmoid_f(z.z + b.z) * p.inv_tau); o.w = expf(logsigmoid_f(z.w + b.w) * p.inv_tau);
+        }
+      } else if (i < dim) {
+        const float f = sec == 0 ? p.q_scale : p.k_scale;
+        const T* src = sec == 0 ? (const T*)p.q + t * p.ldq : (const T*)p.k + t * p.ldk;
+        load_vec<T, 4>(src, false, h * dim + i, x);
+        o = make_float4(x[0] * f, x[1] * f, x[2] * f, x[3] * f);
+      }
+      float* dst = sec == 0 ? w.q : (sec == 1 ? w.k : w.g);
+      *reinterpret_cast<float4*>(dst + (t * p.heads + h) * w.DK + i) = o;
+    } else {
+      const int r = it - 3 * nq, h = r / vq, c = r % vq * 4;
+      if (c < p.vdim) {
+        load_vec<T, 4>((const T*)p.v + t * p.ldv, false, h * p.vdim + c, x);
+        o = make_float4(x[0], x[1], x[2], x[3]);
+      }
+      *reinterpret_cast<float4*>(w.v + (t * p.heads + h) * w.VP + c) = o;
+    }
+  }
+}
+
 // Matrix memory with exponential gates, the scalar side: one warp per (sequence, head) walks the portion's tokens with the
 // running maximum m and the normaliser n (rows spread over the lanes): m' = max(f + m, i); decay = exp(f + m - m'),
 // write = exp(i - m'); n <- decay n + write k; read-out factor = 1 / (max(|n . q|, exp(-m')) + 1e-6).  The three replace
@@ -432,31 +482,42 @@ __global__ void __launch_bounds__(128) exp_gate_kernel(ScanParams p, ScanWork w,
 }
 
 template <int DK, int MODE>
-__global__ void __launch_bounds__(128, DK > 128 ? 2 : 4) state_scan_kernel(ScanParams p, ScanWork w) {
-  constexpr int RP = DK / SCAN_PARTS;  // rows per lane
-  constexpr int RPP = RP + 4;          // a lane's rows start 4 floats further: the four 16-byte reads of a warp hit
-  constexpr int DKP = SCAN_PARTS * RPP;  // different banks
+__global__ void __launch_bounds__(ScanTile<DK>::THREADS) state_scan_kernel(ScanParams p, ScanWork w) {
+  constexpr int PARTS = ScanTile<DK>::PARTS, RP = ScanTile<DK>::RP, RPP = ScanTile<DK>::RPP, DKP = ScanTile<DK>::DKP;
+  constexpr int THREADS = ScanTile<DK>::THREADS;
   constexpr bool ROWS = MODE == SCAN_DELTA || MODE == SCAN_ROWS;        // decay rows beside q and k
   constexpr int NROW = ROWS ? 3 : 2;
-  constexpr int STAGE = SCAN_TOK_TILE * (NROW * DKP + SCAN_COLS + 4);     // floats per stage
+  constexpr int STAGE = SCAN_TOK_TILE * (NROW * DKP + SCAN_COLS + 4);   // floats per stage
+  constexpr int NTOK = PARTS / SCAN_CPL;                                // tokens whose sums are exchanged together
+  constexpr unsigned ALL = 0xffffffffu;
   extern __shared__ __align__(16) float scan_smem[];
   const int vblocks = w.VP / SCAN_COLS;
   const int h = blockIdx.x / vblocks, vb = blockIdx.x % vblocks;
   const int s = blockIdx.y;
   const int t0 = p.cu_q[s], t1 = p.cu_q[s + 1];
   if (t0 >= t1) return;
-  const int part = threadIdx.x % SCAN_PARTS;
-  const int col = threadIdx.x / SCAN_PARTS;
-  const int j = vb * SCAN_COLS + col;
-  const bool active = j < p.vdim;
+  const int part = threadIdx.x % PARTS;
+  const int c0 = threadIdx.x / PARTS * SCAN_CPL;               // first of the lane's columns inside the CTA's block
+  const int j0 = vb * SCAN_COLS + c0;
   const int hk = h / (p.heads / p.qk_heads);
   const int dim = p.dim, vdim = p.vdim;
   const int r0 = part * RP, r0p = part * RPP;
   float* Sg = p.state + ((int64_t)p.slots[s] * p.heads + h) * dim * vdim;
-  float S[RP];
+  const bool vec = vdim % 4 == 0 && j0 < vdim;                 // whole quads of columns, 16-byte aligned
   const bool carried = p.ctx_len[s] > 0;
+  float S[RP][SCAN_CPL];
 #pragma unroll
-  for (int i = 0; i < RP; ++i) S[i] = (carried && active && r0 + i < dim) ? Sg[(int64_t)(r0 + i) * vdim + j] : 0.f;
+  for (int i = 0; i < RP; ++i) {
+    const bool row = carried && r0 + i < dim;
+    const float* src = Sg + (int64_t)(r0 + i) * vdim + j0;
+    if (vec) {
+      const float4 x = row ? *reinterpret_cast<const float4*>(src) : make_float4(0.f, 0.f, 0.f, 0.f);
+      S[i][0] = x.x; S[i][1] = x.y; S[i][2] = x.z; S[i][3] = x.w;
+    } else {
+#pragma unroll
+      for (int c = 0; c < SCAN_CPL; ++c) S[i][c] = (row && j0 + c < vdim) ? src[c] : 0.f;
+    }
+  }
   const float hd = MODE == SCAN_DECAY ? p.head_decay[h] : 0.f;
   const float skip = (MODE == SCAN_GATED && p.head_decay != nullptr) ? p.head_decay[h] : 0.f;
 
@@ -464,16 +525,16 @@ __global__ void __launch_bounds__(128, DK > 128 ? 2 : 4) state_scan_kernel(ScanP
     float* base = scan_smem + stage * STAGE;
     const int nt = min(SCAN_TOK_TILE, t1 - tb);
     constexpr int CH = DK / 4;
-    for (int idx = threadIdx.x; idx < nt * CH; idx += blockDim.x) {
+    for (int idx = threadIdx.x; idx < nt * CH; idx += THREADS) {
       const int tt = idx / CH, c = (idx % CH) * 4;
-      const int dst = tt * DKP + c + 4 * (c / RP);
+      const int dst = tt * DKP + c / RP * RPP + c % RP;
       const int64_t t = tb + tt;
       cp_async16f(base + dst, w.q + (t * p.qk_heads + hk) * DK + c);
       cp_async16f(base + SCAN_TOK_TILE * DKP + dst, w.k + (t * p.qk_heads + hk) * DK + c);
       if (ROWS) cp_async16f(base + 2 * SCAN_TOK_TILE * DKP + dst, w.g + (t * p.heads + h) * DK + c);
     }
     float* sv = base + NROW * SCAN_TOK_TILE * DKP;
-    for (int idx = threadIdx.x; idx < nt * (SCAN_COLS / 4); idx += blockDim.x) {
+    for (int idx = threadIdx.x; idx < nt * (SCAN_COLS / 4); idx += THREADS) {
       const int tt = idx / (SCAN_COLS / 4), c = (idx % (SCAN_COLS / 4)) * 4;
       cp_async16f(sv + tt * SCAN_COLS + c, w.v + ((int64_t)(tb + tt) * p.heads + h) * w.VP + vb * SCAN_COLS + c);
     }
@@ -483,6 +544,19 @@ __global__ void __launch_bounds__(128, DK > 128 ? 2 : 4) state_scan_kernel(ScanP
       cp_async16f(sv + SCAN_TOK_TILE * SCAN_COLS + threadIdx.x * 4,
                   w.gw + ((int64_t)(tb + threadIdx.x) * p.heads + h) * 4);
     asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  // Sums over the lanes of a column group.  `fold` leaves column (part & 3) of a lane's four partial sums joined over its
+  // quad of lanes: (part 0 + part 1) + (part 2 + part 3); quads are joined afterwards in ascending order.
+  const bool b0 = part & 1, b1 = part & 2;
+  auto fold = [&](const float (&o)[SCAN_CPL]) -> float {
+    const float x = (b0 ? o[1] : o[0]) + __shfl_xor_sync(ALL, b0 ? o[0] : o[1], 1);      // column part & 1
+    const float y = (b0 ? o[3] : o[2]) + __shfl_xor_sync(ALL, b0 ? o[2] : o[3], 1);      // column 2 + (part & 1)
+    return (b1 ? y : x) + __shfl_xor_sync(ALL, b1 ? x : y, 2);
+  };
+  auto join_quads = [&](float v) -> float {
+    if (PARTS >= 8) v += __shfl_xor_sync(ALL, v, 4);
+    if (PARTS >= 16) v += __shfl_xor_sync(ALL, v, 8);
+    return v;
   };
 
   load_tile(0, t0);
@@ -501,91 +575,107 @@ __global__ void __launch_bounds__(128, DK > 128 ? 2 : 4) state_scan_kernel(ScanP
     const float* sg = sk + SCAN_TOK_TILE * DKP;
     const float* sv = sq + NROW * SCAN_TOK_TILE * DKP;
     const float* sbeta = sv + SCAN_TOK_TILE * SCAN_COLS;
-    for (int tt = 0; tt < nt; ++tt) {            // every lane takes part in the shuffles, also for a padded column
-      const int64_t t = tb + tt;
-      const float vv = sv[tt * SCAN_COLS + col];
+    // one token: the lane's part of S is advanced; returns column (part & 3) of the read-out joined over the lane's quad
+    auto advance = [&](int tt) -> float {
+      const float4 v4 = *reinterpret_cast<const float4*>(sv + tt * SCAN_COLS + c0);
+      float u[SCAN_CPL] = {v4.x, v4.y, v4.z, v4.w};
       const float* kq = sk + tt * DKP + r0p;
       const float* qq = sq + tt * DKP + r0p;
-      float o0 = 0.f, o1 = 0.f;
-      float4 gwv = make_float4(0.f, 0.f, 1.f, 0.f);
+      const float* gq = sg + tt * DKP + r0p;
+      float dec = hd;
       if (MODE == SCAN_GATED) {
-        gwv = *reinterpret_cast<const float4*>(sbeta + tt * 4);
-        const float u = gwv.y * vv;
+        dec = sbeta[tt * 4];
+        const float wr = sbeta[tt * 4 + 1];
 #pragma unroll
-        for (int i = 0; i < RP; i += 4) {
-          const float4 k4 = *reinterpret_cast<const float4*>(kq + i);
-          const float4 q4 = *reinterpret_cast<const float4*>(qq + i);
-          S[i] = fmaf(gwv.x, S[i], k4.x * u); S[i + 1] = fmaf(gwv.x, S[i + 1], k4.y * u);
-          S[i + 2] = fmaf(gwv.x, S[i + 2], k4.z * u); S[i + 3] = fmaf(gwv.x, S[i + 3], k4.w * u);
-          o0 = fmaf(S[i], q4.x, o0); o1 = fmaf(S[i + 1], q4.y, o1);
-          o0 = fmaf(S[i + 2], q4.z, o0); o1 = fmaf(S[i + 3], q4.w, o1);
-        }
-      } else if (MODE == SCAN_DELTA) {
-        const float* gq = sg + tt * DKP + r0p;
-        float a0 = 0.f, a1 = 0.f;
-#pragma unroll
-        for (int i = 0; i < RP; i += 4) {
-          const float4 g4 = *reinterpret_cast<const float4*>(gq + i);
-          const float4 k4 = *reinterpret_cast<const float4*>(kq + i);
-          S[i] *= g4.x; S[i + 1] *= g4.y; S[i + 2] *= g4.z; S[i + 3] *= g4.w;
-          a0 = fmaf(S[i], k4.x, a0); a1 = fmaf(S[i + 1], k4.y, a1);
-          a0 = fmaf(S[i + 2], k4.z, a0); a1 = fmaf(S[i + 3], k4.w, a1);
-        }
-        float kv = a0 + a1;
-        kv += __shfl_xor_sync(0xffffffffu, kv, 1);
-        kv += __shfl_xor_sync(0xffffffffu, kv, 2);
-        const float u = sbeta[tt] * (vv - kv);
-#pragma unroll
-        for (int i = 0; i < RP; i += 4) {
-          const float4 k4 = *reinterpret_cast<const float4*>(kq + i);
-          const float4 q4 = *reinterpret_cast<const float4*>(qq + i);
-          S[i] = fmaf(k4.x, u, S[i]); S[i + 1] = fmaf(k4.y, u, S[i + 1]);
-          S[i + 2] = fmaf(k4.z, u, S[i + 2]); S[i + 3] = fmaf(k4.w, u, S[i + 3]);
-          o0 = fmaf(S[i], q4.x, o0); o1 = fmaf(S[i + 1], q4.y, o1);
-          o0 = fmaf(S[i + 2], q4.z, o0); o1 = fmaf(S[i + 3], q4.w, o1);
-        }
-      } else if (MODE == SCAN_ROWS) {
-        const float* gq = sg + tt * DKP + r0p;
-#pragma unroll
-        for (int i = 0; i < RP; i += 4) {
-          const float4 g4 = *reinterpret_cast<const float4*>(gq + i);
-          const float4 k4 = *reinterpret_cast<const float4*>(kq + i);
-          const float4 q4 = *reinterpret_cast<const float4*>(qq + i);
-          S[i] = fmaf(g4.x, S[i], k4.x * vv); S[i + 1] = fmaf(g4.y, S[i + 1], k4.y * vv);
-          S[i + 2] = fmaf(g4.z, S[i + 2], k4.z * vv); S[i + 3] = fmaf(g4.w, S[i + 3], k4.w * vv);
-          o0 = fmaf(S[i], q4.x, o0); o1 = fmaf(S[i + 1], q4.y, o1);
-          o0 = fmaf(S[i + 2], q4.z, o0); o1 = fmaf(S[i + 3], q4.w, o1);
-        }
-      } else {
-#pragma unroll
-        for (int i = 0; i < RP; i += 4) {
-          const float4 k4 = *reinterpret_cast<const float4*>(kq + i);
-          const float4 q4 = *reinterpret_cast<const float4*>(qq + i);
-          S[i] = fmaf(hd, S[i], k4.x * vv); S[i + 1] = fmaf(hd, S[i + 1], k4.y * vv);
-          S[i + 2] = fmaf(hd, S[i + 2], k4.z * vv); S[i + 3] = fmaf(hd, S[i + 3], k4.w * vv);
-          o0 = fmaf(S[i], q4.x, o0); o1 = fmaf(S[i + 1], q4.y, o1);
-          o0 = fmaf(S[i + 2], q4.z, o0); o1 = fmaf(S[i + 3], q4.w, o1);
-        }
+        for (int c = 0; c < SCAN_CPL; ++c) u[c] *= wr;
       }
-      float o = o0 + o1;
-      o += __shfl_xor_sync(0xffffffffu, o, 1);
-      o += __shfl_xor_sync(0xffffffffu, o, 2);
-      if (MODE == SCAN_GATED) o = fmaf(o, gwv.z, skip * vv);
-      if (active && part == 0) p.out[t * ((int64_t)p.heads * vdim) + h * vdim + j] = o;
+      if (MODE == SCAN_DELTA) {
+        float a[SCAN_CPL] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+        for (int i = 0; i < RP; i += 4) {
+          const float4 g4 = *reinterpret_cast<const float4*>(gq + i);
+          const float4 k4 = *reinterpret_cast<const float4*>(kq + i);
+          const float gr[4] = {g4.x, g4.y, g4.z, g4.w}, kr[4] = {k4.x, k4.y, k4.z, k4.w};
+#pragma unroll
+          for (int e = 0; e < 4; ++e)
+#pragma unroll
+            for (int c = 0; c < SCAN_CPL; ++c) {
+              S[i + e][c] *= gr[e];
+              a[c] = fmaf(S[i + e][c], kr[e], a[c]);
+            }
+        }
+        // every lane of a column group corrects one column, then collects the quad's four
+        const float mine = sbeta[tt] * (sv[tt * SCAN_COLS + c0 + (part & 3)] - join_quads(fold(a)));
+        const float nb = __shfl_xor_sync(ALL, mine, 1);
+        const float lo = b0 ? nb : mine, hi = b0 ? mine : nb;
+        const float xl = __shfl_xor_sync(ALL, lo, 2), xh = __shfl_xor_sync(ALL, hi, 2);
+        u[0] = b1 ? xl : lo; u[1] = b1 ? xh : hi; u[2] = b1 ? lo : xl; u[3] = b1 ? hi : xh;
+      }
+      float o[SCAN_CPL] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+      for (int i = 0; i < RP; i += 4) {
+        const float4 k4 = *reinterpret_cast<const float4*>(kq + i);
+        const float4 q4 = *reinterpret_cast<const float4*>(qq + i);
+        const float4 g4 = MODE == SCAN_ROWS ? *reinterpret_cast<const float4*>(gq + i) : make_float4(dec, dec, dec, dec);
+        const float gr[4] = {g4.x, g4.y, g4.z, g4.w}, kr[4] = {k4.x, k4.y, k4.z, k4.w}, qr[4] = {q4.x, q4.y, q4.z, q4.w};
+#pragma unroll
+        for (int e = 0; e < 4; ++e)
+#pragma unroll
+          for (int c = 0; c < SCAN_CPL; ++c) {
+            S[i + e][c] = MODE == SCAN_DELTA ? fmaf(kr[e], u[c], S[i + e][c]) : fmaf(gr[e], S[i + e][c], kr[e] * u[c]);
+            o[c] = fmaf(S[i + e][c], qr[e], o[c]);
+          }
+      }
+      return fold(o);
+    };
+    auto emit = [&](int tt, float o) {           // column (part & 3) of token tt's read-out
+      if (MODE == SCAN_GATED) o = fmaf(o, sbeta[tt * 4 + 2], skip * sv[tt * SCAN_COLS + c0 + (part & 3)]);
+      const int j = j0 + (part & 3);
+      if (j < vdim) p.out[(int64_t)(tb + tt) * ((int64_t)p.heads * vdim) + h * vdim + j] = o;
+    };
+    // NTOK tokens at a time: only S ties them together, so their loads and sums overlap; the quads exchange their sums so
+    // that quad n ends up with token n's total (the same pairs in the same order as one token alone takes: the result does
+    // not depend on how a portion falls into groups)
+    int tt = 0;
+#pragma unroll 2
+    for (; tt + NTOK <= nt; tt += NTOK) {        // every lane takes part in the shuffles, also for a padded column
+      float v[NTOK];
+#pragma unroll
+      for (int n = 0; n < NTOK; ++n) v[n] = advance(tt + n);
+      if (NTOK == 4) {
+        const bool q0 = part & 4, q1 = part & 8;
+        const float x = (q0 ? v[1 % NTOK] : v[0]) + __shfl_xor_sync(ALL, q0 ? v[0] : v[1 % NTOK], 4);
+        const float y = (q0 ? v[3 % NTOK] : v[2 % NTOK]) + __shfl_xor_sync(ALL, q0 ? v[2 % NTOK] : v[3 % NTOK], 4);
+        v[0] = (q1 ? y : x) + __shfl_xor_sync(ALL, q1 ? x : y, 8);
+      } else if (NTOK == 2) {
+        const bool q0 = part & 4;
+        v[0] = (q0 ? v[1 % NTOK] : v[0]) + __shfl_xor_sync(ALL, q0 ? v[0] : v[1 % NTOK], 4);
+      }
+      emit(tt + part / SCAN_CPL, v[0]);
+    }
+    for (; tt < nt; ++tt) {
+      const float o = join_quads(advance(tt));
+      if (part < SCAN_CPL) emit(tt, o);
     }
     __syncthreads();                            // this stage may be refilled in the next pass
   }
-  if (active) {
 #pragma unroll
-    for (int i = 0; i < RP; ++i)
-      if (r0 + i < dim) Sg[(int64_t)(r0 + i) * vdim + j] = S[i];
-  }
+  for (int i = 0; i < RP; ++i)
+    if (r0 + i < dim) {
+      float* dst = Sg + (int64_t)(r0 + i) * vdim + j0;
+      if (vec) {
+        *reinterpret_cast<float4*>(dst) = make_float4(S[i][0], S[i][1], S[i][2], S[i][3]);
+      } else {
+#pragma unroll
+        for (int c = 0; c < SCAN_CPL; ++c)
+          if (j0 + c < vdim) dst[c] = S[i][c];
+      }
+    }
 }
 
 template <int DK, int MODE> int launch_scan_dk(const ScanParams& p, const ScanWork& w, int nseq, cudaStream_t st) {
-  constexpr int DKP = SCAN_PARTS * (DK / SCAN_PARTS + 4);
   constexpr int NROW = MODE == SCAN_DELTA || MODE == SCAN_ROWS ? 3 : 2;
-  const size_t smem = (size_t)2 * SCAN_TOK_TILE * (NROW * DKP + SCAN_COLS + 4) * sizeof(float);
+  const size_t smem = (size_t)2 * SCAN_TOK_TILE * (NROW * ScanTile<DK>::DKP + SCAN_COLS + 4) * sizeof(float);
   auto kern = state_scan_kernel<DK, MODE>;
   static bool configured = false;
   if (!configured) {
@@ -594,7 +684,7 @@ template <int DK, int MODE> int launch_scan_dk(const ScanParams& p, const ScanWo
     configured = true;
   }
   dim3 grid(p.heads * (w.VP / SCAN_COLS), nseq);
-  kern<<<grid, SCAN_COLS * SCAN_PARTS, smem, st>>>(p, w);
+  kern<<<grid, ScanTile<DK>::THREADS, smem, st>>>(p, w);
   return CB_LAUNCH_CHECK();
 }
 
@@ -614,7 +704,13 @@ int launch_scan(const ScanParams& p, float* work, int64_t tokens, int nseq, cuda
   w.beta = w.g + (MODE == SCAN_DELTA || MODE == SCAN_ROWS ? tokens * p.heads * w.DK : 0);
   w.gw = w.beta;
   w.v = w.beta + (MODE == SCAN_DELTA ? (tokens * p.heads + 3) / 4 * 4 : (MODE == SCAN_GATED ? tokens * p.heads * 4 : 0));
-  scan_prepare_kernel<MODE, T><<<(unsigned)tokens, 128, 0, st>>>(p, w);
+  auto quads = [](const void* q, int64_t ld, size_t es) { return ld % 4 == 0 && ((uintptr_t)q % (4 * es)) == 0; };
+  if (MODE == SCAN_ROWS && !p.act_silu && !p.unit_qk && p.rot_table == nullptr && p.heads == p.qk_heads && p.dim % 4 == 0 &&
+      p.vdim % 4 == 0 && quads(p.q, p.ldq, sizeof(T)) && quads(p.k, p.ldk, sizeof(T)) && quads(p.v, p.ldv, sizeof(T)) &&
+      quads(p.araw, p.lda, 4) && quads(p.dt_bias, 0, 4) && quads(work, 0, 4))
+    scan_prepare_rows_vec_kernel<T><<<(unsigned)tokens, 256, 0, st>>>(p, w);
+  else
+    scan_prepare_kernel<MODE, T><<<(unsigned)tokens, 128, 0, st>>>(p, w);
   if (MODE == SCAN_GATED && p.gate_kind == GATE_EXP) {
     const unsigned blocks = (unsigned)((nseq * p.heads + 3) / 4);
     if (w.DK == 16) exp_gate_kernel<16><<<blocks, 128, 0, st>>>(p, w, nseq);
@@ -2396,7 +2492,7 @@ __global__ void __launch_bounds__(256) rotary_kv_write_kernel(T* __restrict__ qk
 // position and divided by sqrt(mean of squares + eps); queries go to q_out, keys and values into their pages.  fp32 from the
 // first load to the one rounding at the store.  A lane holds VEC adjacent channels per step, ITEMS steps; the head sits in
 // shared memory while it is turned.
-constexpr int CRW_TOK_TILE = 16;
+constexpr int CRW_TOK_TILE = 32, CRW_AHEAD = 4;
 
 template <typename T> struct ConvRotArgs {
   const T *x, *w, *state;
@@ -2409,7 +2505,7 @@ template <typename T> struct ConvRotArgs {
 };
 
 template <typename T, int VEC, int ITEMS, int TAPS>
-__global__ void __launch_bounds__(128) conv_rotary_kv_write_kernel(ConvRotArgs<T> a) {
+__global__ void __launch_bounds__(128, VEC == 4 && ITEMS == 1 ? 6 : 1) conv_rotary_kv_write_kernel(ConvRotArgs<T> a) {
   struct alignas(sizeof(T) * VEC) Pack { T v[VEC]; };
   extern __shared__ __align__(16) float crw_smem[];
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -2448,80 +2544,121 @@ __global__ void __launch_bounds__(128) conv_rotary_kv_write_kernel(ConvRotArgs<T
   }
   float* sm = crw_smem + warp * (ITEMS * 32 * VEC);
   const int half = a.rot >> 1;
+  // whole vectors of partners: neighbours sit in the lane's own registers, the other half of the head in one 16-byte read
+  const bool wide = VEC == 4 && (a.interleaved ? a.rot % 8 == 0 : half % 4 == 0);
   const int j1 = min(j0 + CRW_TOK_TILE, qlen);
-  for (int j = j0; j < j1; ++j) {
-    const int pos = ctx + j;
-    float y[ITEMS][VEC];
+  for (int jb = j0; jb < j1; jb += CRW_AHEAD) {
+    Pack in[CRW_AHEAD][ITEMS];                               // the rows of several tokens are in flight at once
 #pragma unroll
-    for (int it = 0; it < ITEMS; ++it) {
-      const int c = (lane + 32 * it) * VEC;
-      if (c < width) {
-        const Pack p = *reinterpret_cast<const Pack*>(xr + (int64_t)j * a.ldx + c);
+    for (int n = 0; n < CRW_AHEAD; ++n)
 #pragma unroll
-        for (int e = 0; e < VEC; ++e) {
-          const float cur = to_f32<T>(p.v[e]);
-          float acc = 0.f;
-#pragma unroll
-          for (int i = 0; i < TAPS - 1; ++i) acc = fmaf(wt[it][i][e], win[it][i][e], acc);
-          y[it][e] = fmaf(wt[it][TAPS - 1][e], cur, acc);
-#pragma unroll
-          for (int i = 0; i < TAPS - 2; ++i) win[it][i][e] = win[it][i + 1][e];
-          if (TAPS > 1) win[it][TAPS > 1 ? TAPS - 2 : 0][e] = cur;
-        }
+      for (int it = 0; it < ITEMS; ++it) {
+        const int c = (lane + 32 * it) * VEC;
+        if (c < width && jb + n < j1) in[n][it] = *reinterpret_cast<const Pack*>(xr + (int64_t)(jb + n) * a.ldx + c);
       }
-    }
-    if (!value && a.rot > 0) {
-      __syncwarp();                                          // the last token's partners have been read
 #pragma unroll
-      for (int it = 0; it < ITEMS; ++it)
+    for (int n = 0; n < CRW_AHEAD; ++n) {
+      const int j = jb + n, pos = ctx + j;
+      if (j >= j1) break;
+      float y[ITEMS][VEC];
 #pragma unroll
-        for (int e = 0; e < VEC; ++e) sm[(lane + 32 * it) * VEC + e] = y[it][e];
-      __syncwarp();
-      const float* cs = a.table + (int64_t)pos * a.rot;
-#pragma unroll
-      for (int it = 0; it < ITEMS; ++it)
-#pragma unroll
-        for (int e = 0; e < VEC; ++e) {
-          const int c = (lane + 32 * it) * VEC + e;
-          if (c < a.rot) {                                   // pair index, partner, and which half of the pair this is
-            const int pi = a.interleaved ? c >> 1 : (c < half ? c : c - half);
-            const int pc = a.interleaved ? c ^ 1 : (c < half ? c + half : c - half);
-            const bool first = a.interleaved ? !(c & 1) : c < half;
-            const float sn = cs[half + pi];
-            y[it][e] = fmaf(y[it][e], cs[pi], first ? -sm[pc] * sn : sm[pc] * sn);
-          }
-        }
-    }
-    if (!value && a.unit) {
-      float ss = 0.f;
-#pragma unroll
-      for (int it = 0; it < ITEMS; ++it)
+      for (int it = 0; it < ITEMS; ++it) {
         if ((lane + 32 * it) * VEC < width) {
 #pragma unroll
-          for (int e = 0; e < VEC; ++e) ss = fmaf(y[it][e], y[it][e], ss);
+          for (int e = 0; e < VEC; ++e) {
+            const float cur = to_f32<T>(in[n][it].v[e]);
+            float acc = 0.f;
+#pragma unroll
+            for (int i = 0; i < TAPS - 1; ++i) acc = fmaf(wt[it][i][e], win[it][i][e], acc);
+            y[it][e] = fmaf(wt[it][TAPS - 1][e], cur, acc);
+#pragma unroll
+            for (int i = 0; i < TAPS - 2; ++i) win[it][i][e] = win[it][i + 1][e];
+            if (TAPS > 1) win[it][TAPS > 1 ? TAPS - 2 : 0][e] = cur;
+          }
         }
-      const float r = 1.f / sqrtf(warp_sum(ss) / (float)width + a.eps);
+      }
+      if (!value && a.rot > 0) {
+        const float* cs = a.table + (int64_t)pos * a.rot;
+        if (!(wide && a.interleaved)) {
+          __syncwarp();                                      // the last token's partners have been read
 #pragma unroll
-      for (int it = 0; it < ITEMS; ++it)
+          for (int it = 0; it < ITEMS; ++it) {
+            float* d = sm + (lane + 32 * it) * VEC;
+            if (VEC == 4) *reinterpret_cast<float4*>(d) = make_float4(y[it][0], y[it][VEC > 1 ? 1 : 0], y[it][VEC > 2 ? 2 : 0],
+                                                                      y[it][VEC > 3 ? 3 : 0]);
+            else d[0] = y[it][0];
+          }
+          __syncwarp();
+        }
 #pragma unroll
-        for (int e = 0; e < VEC; ++e) y[it][e] *= r;
-    }
-    T* dst;
-    if (unit < a.H) {
-      dst = a.q_out + ((int64_t)(t0 + j) * a.H + unit) * a.dim;
-    } else {
-      const int64_t row = (int64_t)a.block_tables[(int64_t)s * a.max_blocks + pos / a.block_size] * a.block_size +
-                          pos % a.block_size;
-      dst = value ? a.v_cache + (row * a.G + unit - a.H - a.G) * a.vdim : a.k_cache + (row * a.G + unit - a.H) * a.dim;
-    }
+        for (int it = 0; it < ITEMS; ++it) {
+          const int c = (lane + 32 * it) * VEC;
+          if (c >= a.rot) continue;
+          if (wide) {
+            if (a.interleaved) {
+              const float2 co = *reinterpret_cast<const float2*>(cs + (c >> 1));
+              const float2 sn = *reinterpret_cast<const float2*>(cs + half + (c >> 1));
+              const float u0 = y[it][0], v0 = y[it][VEC > 1 ? 1 : 0], u1 = y[it][VEC > 2 ? 2 : 0], v1 = y[it][VEC > 3 ? 3 : 0];
+              y[it][0] = u0 * co.x - v0 * sn.x;
+              y[it][VEC > 1 ? 1 : 0] = v0 * co.x + u0 * sn.x;
+              y[it][VEC > 2 ? 2 : 0] = u1 * co.y - v1 * sn.y;
+              y[it][VEC > 3 ? 3 : 0] = v1 * co.y + u1 * sn.y;
+            } else {
+              const bool first = c < half;
+              const int pi = first ? c : c - half;
+              const float4 o = *reinterpret_cast<const float4*>(sm + (first ? c + half : c - half));
+              const float4 co = *reinterpret_cast<const float4*>(cs + pi), sn = *reinterpret_cast<const float4*>(cs + half + pi);
+              const float sg = first ? -1.f : 1.f;
+              const float ov[4] = {o.x, o.y, o.z, o.w}, cv[4] = {co.x, co.y, co.z, co.w}, sv[4] = {sn.x, sn.y, sn.z, sn.w};
 #pragma unroll
-    for (int it = 0; it < ITEMS; ++it) {
-      const int c = (lane + 32 * it) * VEC;
-      if (c < width) {
-        Pack p;
+              for (int e = 0; e < VEC; ++e) y[it][e] = fmaf(y[it][e], cv[e], sg * ov[e] * sv[e]);
+            }
+            continue;
+          }
 #pragma unroll
-        for (int e = 0; e < VEC; ++e) p.v[e] = from_f32<T>(y[it][e]);
-        *reinterpret_cast<Pack*>(dst + c) = p;
+          for (int e = 0; e < VEC; ++e) {
+            const int ce = c + e;
+            if (ce < a.rot) {                                // pair index, partner, and which half of the pair this is
+              const int pi = a.interleaved ? ce >> 1 : (ce < half ? ce : ce - half);
+              const int pc = a.interleaved ? ce ^ 1 : (ce < half ? ce + half : ce - half);
+              const bool first = a.interleaved ? !(ce & 1) : ce < half;
+              const float sn = cs[half + pi];
+              y[it][e] = fmaf(y[it][e], cs[pi], first ? -sm[pc] * sn : sm[pc] * sn);
+            }
+          }
+        }
+      }
+      if (!value && a.unit) {
+        float ss = 0.f;
+#pragma unroll
+        for (int it = 0; it < ITEMS; ++it)
+          if ((lane + 32 * it) * VEC < width) {
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) ss = fmaf(y[it][e], y[it][e], ss);
+          }
+        const float r = 1.f / sqrtf(warp_sum(ss) / (float)width + a.eps);
+#pragma unroll
+        for (int it = 0; it < ITEMS; ++it)
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) y[it][e] *= r;
+      }
+      T* dst;
+      if (unit < a.H) {
+        dst = a.q_out + ((int64_t)(t0 + j) * a.H + unit) * a.dim;
+      } else {
+        const int64_t row = (int64_t)a.block_tables[(int64_t)s * a.max_blocks + pos / a.block_size] * a.block_size +
+                            pos % a.block_size;
+        dst = value ? a.v_cache + (row * a.G + unit - a.H - a.G) * a.vdim : a.k_cache + (row * a.G + unit - a.H) * a.dim;
+      }
+#pragma unroll
+      for (int it = 0; it < ITEMS; ++it) {
+        const int c = (lane + 32 * it) * VEC;
+        if (c < width) {
+          Pack p;
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) p.v[e] = from_f32<T>(y[it][e]);
+          *reinterpret_cast<Pack*>(dst + c) = p;
+        }
       }
     }
   }
